@@ -1,16 +1,20 @@
 // Softmax attention over the paged cache with a sliding window behind which whole blocks of tokens stay in sight as one
 // pooled key and value each, a sink per head in the softmax's denominator, a query multiplier that grows with the
-// position, and values that may be the keys themselves.  Every one of these is optional, so the same kernels serve plain
-// causal attention whose values are its keys and windowed attention with pooled blocks.
+// position, values that may be the keys themselves, capped scores and a gate per head.  Every one of these is optional, so the
+// same kernels serve plain causal attention whose values are its keys, windowed attention with pooled blocks, and causal
+// attention with capped scores, a sink and gated heads.
 //
 // Row i of a sequence sees token j if 0 <= i - j < window (window 0: every j <= i), and pooled block b (positions
 // b P .. b P + P - 1) if b P + P - 1 <= i - window: the first floor(max(0, i - window + 1) / P) blocks.  Tokens and blocks
 // share one softmax; with a sink s_h the denominator also holds exp(s_h).  Head h's scores are (q . k) * scale * m(i) with
-// m(i) = 1 + coef * ln(floor((i + 1) / every) + 1), the multiplier applied to the 32-bit score, not to the stored query.
+// m(i) = 1 + coef * ln(floor((i + 1) / every) + 1), the multiplier applied to the 32-bit score, not to the stored query; with a cap
+// c a score s becomes c tanh(s / c).  Head h's result is multiplied by sigmoid(gate_h) where the rows carry gates.
 //
 //   prepare   per row: q and k heads are RMS-normed with a weight shared by the heads (optional), the first `rot` numbers
 //             of each head turn by position (pairs (i, i + rot / 2), angle fp32(pos) * freq[i], cosine and sine times a
-//             multiplier; optional); q goes back in place, k and v go to the cache rows of (sequence, position).
+//             multiplier; optional); q goes back in place, k and v go to the cache rows of (sequence, position).  The pairs may
+//             be (2i, 2i + 1) instead; prepare_whole norms all query heads of a row as one vector (weights [heads * dim]), likewise
+//             the key heads, a block per row.
 //   pool      the block sums: pooled row b of a sequence holds the SUM of the block's keys (and values) as the cache keeps
 //             them, in 32-bit, added token by token in the order of positions whatever the steps were (a block that a step
 //             continues starts from what the steps before left); readers multiply by 1 / P.  Pooled rows are paged like
@@ -35,6 +39,8 @@ constexpr int PAGE_ROWS = 64;
 __device__ __forceinline__ float query_multiplier(int pos, float coef, int every) {
     return every > 0 ? 1.0f + coef * logf((float)((pos + 1) / every) + 1.0f) : 1.0f;
 }
+// cap * tanh(s / cap); cap 0: s
+__device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 __device__ __forceinline__ int blocks_in_sight(int pos, int window, int pool) {
     return (pool > 0 && window > 0) ? max(0, pos - window + 1) / pool : 0;
 }
@@ -50,6 +56,7 @@ struct PrepArgs {
     const int* row_seq;
     const int* row_pos;
     int ld, q_off, k_off, v_off, heads, kv_heads, dim, vdim, rot, table_width, rows, write;
+    int neighbours;          // the rotated pairs are (2i, 2i + 1) instead of (i, i + rot / 2)
     float eps, rot_mult;
 };
 
@@ -109,11 +116,146 @@ __global__ void __launch_bounds__(128) prepare_kernel(PrepArgs p) {
         s *= p.rot_mult;
         c *= p.rot_mult;
         float a, b;
-        fr_rotate(buf[i], buf[i + half], c, s, a, b);
-        fr_store(dst + i, a);
-        fr_store(dst + i + half, b);
+        const int i0 = p.neighbours ? 2 * i : i, i1 = p.neighbours ? 2 * i + 1 : i + half;
+        fr_rotate(buf[i0], buf[i1], c, s, a, b);
+        fr_store(dst + i0, a);
+        fr_store(dst + i1, b);
     }
     for (int i = 2 * half + lane; i < p.dim; i += 32) fr_store(dst + i, buf[i]);
+}
+
+// ---- one norm over all query heads of a row, one over its key heads; neighbouring pairs; a block per row
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 a = *(const float4*)p, b = *(const float4*)(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {
+    const uint4 r = *(const uint4*)p;
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
+    *(float4*)p = make_float4(v[0], v[1], v[2], v[3]);
+    *(float4*)(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void store8(bf16* p, const float (&v)[8]) {
+    uint4 r;
+    __nv_bfloat162* h = (__nv_bfloat162*)&r;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *(uint4*)p = r;
+}
+
+constexpr int WHOLE_THREADS = 256;
+
+// `pieces`: heads, offsets and rows are whole runs of eight channels on 16-byte boundaries
+template <typename T>
+__global__ void __launch_bounds__(WHOLE_THREADS) prepare_whole_kernel(PrepArgs p, int pieces) {
+    __shared__ float2 turn[128];              // cosine and sine of the row's angles, shared by the heads
+    __shared__ float part[2][WHOLE_THREADS / 32];
+    const int row = blockIdx.x, seq = p.row_seq[row];
+    fr_pdl_wait();
+    fr_pdl_launch();
+    if (seq < 0) return;
+    const int pos = p.row_pos[row], half = p.freq != nullptr ? p.rot / 2 : 0;
+    for (int i = threadIdx.x; i < half; i += WHOLE_THREADS) {
+        float s, c;
+        sincosf((float)pos * p.freq[i], &s, &c);
+        turn[i] = make_float2(c * p.rot_mult, s * p.rot_mult);
+    }
+    T* x = (T*)p.proj + (size_t)row * p.ld;
+    const int nq = p.heads * p.dim, nk = p.write ? p.kv_heads * p.dim : 0;
+    float sum[2] = {0.f, 0.f};
+    for (int which = 0; which < 2; ++which) {
+        const T* src = x + (which ? p.k_off : p.q_off);
+        const int n = which ? nk : nq;
+        float ss = 0.f;
+        if (pieces) {
+            for (int c = threadIdx.x * 8; c < n; c += WHOLE_THREADS * 8) {
+                float v[8];
+                load8(src + c, v);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
+            }
+        } else {
+            for (int c = threadIdx.x; c < n; c += WHOLE_THREADS) {
+                const float v = fr_load(src + c);
+                ss = fmaf(v, v, ss);
+            }
+        }
+        sum[which] = fr_warp_sum(ss);
+    }
+    if ((threadIdx.x & 31) == 0) {
+        part[0][threadIdx.x >> 5] = sum[0];
+        part[1][threadIdx.x >> 5] = sum[1];
+    }
+    __syncthreads();
+    sum[0] = sum[1] = 0.f;
+    for (int w = 0; w < WHOLE_THREADS / 32; ++w) {
+        sum[0] += part[0][w];
+        sum[1] += part[1][w];
+    }
+    size_t at = 0;
+    if (p.write) at = (size_t)p.block_table[(size_t)seq * p.table_width + pos / PAGE_ROWS] * PAGE_ROWS + pos % PAGE_ROWS;
+    for (int which = 0; which < 2; ++which) {
+        const int n = which ? nk : nq;
+        const T* src = x + (which ? p.k_off : p.q_off);
+        T* dst = which ? (T*)p.k_pool + at * p.kv_heads * p.dim : x + p.q_off;
+        const FrVec& w = which ? p.k_norm : p.q_norm;
+        const float inv = w.p != nullptr ? 1.0f / sqrtf(sum[which] / (float)n + p.eps) : 1.f;
+        if (pieces) {
+            for (int c = threadIdx.x * 8; c < n; c += WHOLE_THREADS * 8) {
+                float v[8];
+                load8(src + c, v);
+                if (w.p != nullptr)
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * w.at(c + i);
+                const int d = c % p.dim;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int pair = d / 2 + i;
+                    if (pair < half) {
+                        const float2 t = turn[pair];
+                        const float a = v[2 * i], b = v[2 * i + 1];
+                        fr_rotate(a, b, t.x, t.y, v[2 * i], v[2 * i + 1]);
+                    }
+                }
+                store8(dst + c, v);
+            }
+        } else {
+            const int per = (p.dim + 1) / 2, items = n / p.dim * per;          // pairs of a head (an odd head ends with one channel)
+            for (int idx = threadIdx.x; idx < items; idx += WHOLE_THREADS) {
+                const int head = idx / per, pair = idx - head * per, c = head * p.dim + 2 * pair;
+                const bool two = 2 * pair + 1 < p.dim;
+                float a = fr_load(src + c), b = two ? fr_load(src + c + 1) : 0.f;
+                if (w.p != nullptr) {
+                    a = a * inv * w.at(c);
+                    if (two) b = b * inv * w.at(c + 1);
+                }
+                if (pair < half) {
+                    const float2 t = turn[pair];
+                    const float a0 = a, b0 = b;
+                    fr_rotate(a0, b0, t.x, t.y, a, b);
+                }
+                fr_store(dst + c, a);
+                if (two) fr_store(dst + c + 1, b);
+            }
+        }
+    }
+    if (p.write && p.v_pool != nullptr) {
+        const int n = p.kv_heads * p.vdim;
+        const T* src = x + p.v_off;
+        T* dst = (T*)p.v_pool + at * n;
+        constexpr int PER = 16 / (int)sizeof(T);
+        if (n % PER == 0 && (((uintptr_t)src | (uintptr_t)dst) & 15) == 0)
+            for (int c = threadIdx.x; c < n / PER; c += WHOLE_THREADS) ((uint4*)dst)[c] = ((const uint4*)src)[c];
+        else
+            for (int c = threadIdx.x; c < n; c += WHOLE_THREADS) dst[c] = src[c];
+    }
 }
 
 // ------------------------------------------------------------------ pool
@@ -180,8 +322,9 @@ struct RowArgs {
     const int* row_pos;
     FrVec sink;              // [heads]; p null: none
     float* part;             // [rows][heads][splits][vdim + 2]
+    const void* gate;        // head h's gate of row r at gate[r * q_stride + h]; null: none
     int table_width, pool_table_width, rows, heads, kv_heads, dim, vdim, q_stride, q_off, window, pool, splits, temp_every;
-    float scale, temp_coef;
+    float scale, temp_coef, softcap;
 };
 
 // `count` keys from index `first` of one source: their rows are at row_of(i); four at a time, loads issued together
@@ -223,7 +366,7 @@ __device__ __forceinline__ void walk(const RowArgs& p, const KT* kbase, const KT
         float m_new = m;
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
-            s4[u] *= kmul;
+            s4[u] = capped(s4[u] * kmul, p.softcap);
             if (i + u < end) m_new = fmaxf(m_new, s4[u]);
         }
         const float alpha = expf(m - m_new);
@@ -317,7 +460,8 @@ __global__ void __launch_bounds__(128) rows_merge_kernel(RowArgs p) {
             if (d < p.vdim) acc[i] += ps[d] * f;
         }
     }
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    float inv = l > 0.f ? 1.0f / l : 0.f;
+    if (p.gate != nullptr) inv /= 1.0f + expf(-fr_load((const T*)p.gate + (size_t)(item / p.heads) * p.q_stride + h));
     T* o_row = (T*)p.out + (size_t)item * p.vdim;
 #pragma unroll
     for (int i = 0; i < MAX_PER_LANE; ++i) {
@@ -342,8 +486,9 @@ struct PromptArgs {
     const int* seq_qlen;
     const int* seq_pos0;
     FrVec sink;
+    const bf16* gate;        // head h's gate of row r at gate[r * q_stride + h]; null: none
     int table_width, pool_table_width, q_stride, q_off, heads, kv_heads, dim, vdim, window, pool, temp_every;
-    float scale, temp_coef;
+    float scale, temp_coef, softcap;
 };
 
 __device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -473,7 +618,7 @@ __global__ void __launch_bounds__(128, 3) prompt_kernel(PromptArgs p) {
                 const int j = b * BN + nt * 8 + 2 * t + (e & 1), half = e >> 1;
                 const int pos = my_pos[half];
                 const bool seen = pos <= last_pos && (pooled ? j < my_blocks[half] : (j <= pos && (p.window <= 0 || pos - j < p.window)));
-                s[nt][e] = seen ? s[nt][e] * mult[half] : -INFINITY;
+                s[nt][e] = seen ? capped(s[nt][e] * mult[half], p.softcap) : -INFINITY;
                 m_new[half] = fmaxf(m_new[half], s[nt][e]);
             }
         }
@@ -537,7 +682,8 @@ __global__ void __launch_bounds__(128, 3) prompt_kernel(PromptArgs p) {
             f = expf(m_run[half] - big);
             l = l * f + expf(sink - big);
         }
-        const float inv = l > 0.f ? f / l : 0.f;
+        float inv = l > 0.f ? f / l : 0.f;
+        if (p.gate != nullptr) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)(row0 + r) * p.q_stride + h]));
         bf16* dst = p.out + (size_t)(row0 + r) * p.heads * p.vdim + (size_t)h * p.vdim;
 #pragma unroll
         for (int nt = 0; nt < DV / 8; ++nt) {
@@ -585,9 +731,11 @@ int check_shape(int heads, int kv_heads, int dim, int vdim, int window, int pool
 
 // proj [rows][ld] of `dtype`: q heads at q_off, k heads at k_off, v heads at v_off (v_pool null: the values are the keys and
 // nothing is read at v_off).  q_norm / k_norm [dim] of norm_dtype (null: no norm); freq [rot / 2] (null: no rotation).
-// write 0: the cache is left alone (queries only).
+// write 0: the cache is left alone (queries only).  neighbours: the rotated pairs are (2i, 2i + 1).  norm_whole: one norm over all
+// query heads (q_norm [heads * dim]) and one over all key heads (k_norm [kv_heads * dim]).
 FR_EXPORT int attention_pooled_prepare(void* proj, int ld, int q_off, int k_off, int v_off, const void* q_norm, const void* k_norm,
-                                       int norm_dtype, float eps, const float* freq, float rot_mult, int rot, void* k_pool, void* v_pool,
+                                       int norm_dtype, float eps, const float* freq, float rot_mult, int rot, int neighbours, int norm_whole,
+                                       void* k_pool, void* v_pool,
                                        const int* block_table, int table_width, int page, const int* row_seq, const int* row_pos, int rows,
                                        int heads, int kv_heads, int dim, int vdim, int write, int dtype, cudaStream_t stream) {
     if (rows <= 0) return FR_OK;
@@ -598,7 +746,17 @@ FR_EXPORT int attention_pooled_prepare(void* proj, int ld, int q_off, int k_off,
     p.proj = proj; p.q_norm = FrVec{q_norm, norm_dtype}; p.k_norm = FrVec{k_norm, norm_dtype}; p.freq = freq; p.k_pool = k_pool; p.v_pool = v_pool;
     p.block_table = block_table; p.row_seq = row_seq; p.row_pos = row_pos; p.ld = ld; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
     p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.rot = rot; p.table_width = table_width; p.rows = rows; p.write = write;
-    p.eps = eps; p.rot_mult = rot_mult;
+    p.eps = eps; p.rot_mult = rot_mult; p.neighbours = neighbours;
+    if (norm_whole) {
+        if (freq != nullptr && (!neighbours || rot > 256)) FR_REFUSE("attention_pooled: a norm over all heads goes with up to 256 rotated numbers in neighbouring pairs");
+        const int off = q_off | k_off | ld | dim;
+        const int pieces = off % 8 == 0 && ((((uintptr_t)proj) | ((uintptr_t)k_pool)) & 15) == 0;
+        if (dtype == FR_F32) FR_CUDA(fr_launch(prepare_whole_kernel<float>, dim3(rows), dim3(WHOLE_THREADS), 0, stream, p, pieces));
+        else if (dtype == FR_BF16) FR_CUDA(fr_launch(prepare_whole_kernel<bf16>, dim3(rows), dim3(WHOLE_THREADS), 0, stream, p, pieces));
+        else FR_REFUSE("attention_pooled: unknown dtype %d", dtype);
+        FR_CHECK_LAUNCH("attention_pooled prepare (whole)");
+        return FR_OK;
+    }
     const long long items = (long long)rows * (heads + 2 * kv_heads);
     const dim3 grid((unsigned)((items + 3) / 4));
     if (dtype == FR_F32) FR_CUDA(fr_launch(prepare_kernel<float>, grid, dim3(128), 0, stream, p));
@@ -633,13 +791,14 @@ FR_EXPORT long long attention_pooled_scratch_floats(int rows, int heads, int vdi
 }
 
 // q [rows][q_stride] and out [rows][heads * vdim] of `dtype`, like the token pools; the pooled pools are fp32 sums (null with
-// pool 0).  sink [heads] of sink_dtype (null: none).  temp_every 0: no query multiplier.
+// pool 0).  sink [heads] of sink_dtype (null: none).  temp_every 0: no query multiplier; softcap 0: none.  gate: head h's gate of
+// row r at gate[r * q_stride + h], in the rows' dtype (null: none).
 FR_EXPORT int attention_pooled_rows(const void* q, int q_stride, int q_off, void* out, const void* k_pool, const void* v_pool,
                                     const float* pk_pool, const float* pv_pool, const int* block_table, int table_width,
                                     const int* pool_table, int pool_table_width, int page, const int* row_seq, const int* row_pos, int rows,
                                     int heads, int kv_heads, int dim, int vdim, int window, int pool, float scale, float temp_coef,
-                                    int temp_every, const void* sink, int sink_dtype, int splits, float* scratch, int dtype,
-                                    cudaStream_t stream) {
+                                    int temp_every, float softcap, const void* sink, int sink_dtype, const void* gate, int splits,
+                                    float* scratch, int dtype, cudaStream_t stream) {
     if (rows <= 0) return FR_OK;
     const int rc = check_shape(heads, kv_heads, dim, vdim, window, pool, page);
     if (rc != FR_OK) return rc;
@@ -650,7 +809,7 @@ FR_EXPORT int attention_pooled_rows(const void* q, int q_stride, int q_off, void
     p.pool_table = pool_table; p.row_seq = row_seq; p.row_pos = row_pos; p.sink = FrVec{sink, sink_dtype}; p.part = scratch;
     p.table_width = table_width; p.pool_table_width = pool_table_width; p.rows = rows; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim;
     p.vdim = vdim; p.q_stride = q_stride; p.q_off = q_off; p.window = window; p.pool = pool; p.splits = splits; p.temp_every = temp_every;
-    p.scale = scale; p.temp_coef = temp_coef;
+    p.scale = scale; p.temp_coef = temp_coef; p.softcap = softcap; p.gate = gate;
     const int items = rows * heads;
     const dim3 grid((items + 3) / 4, splits), mgrid((items + 3) / 4);
     if (dtype == FR_F32) {
@@ -673,8 +832,8 @@ FR_EXPORT int attention_pooled_prompt(const void* q, int q_stride, int q_off, vo
                                       const float* pk_pool, const float* pv_pool, const int* block_table, int table_width,
                                       const int* pool_table, int pool_table_width, int page, const int* seq_start, const int* seq_qlen,
                                       const int* seq_pos0, int n_seqs, int max_q_len, int heads, int kv_heads, int dim, int vdim, int window,
-                                      int pool, float scale, float temp_coef, int temp_every, const void* sink, int sink_dtype,
-                                      cudaStream_t stream) {
+                                      int pool, float scale, float temp_coef, int temp_every, float softcap, const void* sink, int sink_dtype,
+                                      const void* gate, cudaStream_t stream) {
     if (n_seqs <= 0 || max_q_len <= 0) return FR_OK;
     const int rc = check_shape(heads, kv_heads, dim, vdim, window, pool, page);
     if (rc != FR_OK) return rc;
@@ -686,7 +845,7 @@ FR_EXPORT int attention_pooled_prompt(const void* q, int q_stride, int q_off, vo
     p.block_table = block_table; p.pool_table = pool_table; p.seq_start = seq_start; p.seq_qlen = seq_qlen; p.seq_pos0 = seq_pos0;
     p.sink = FrVec{sink, sink_dtype}; p.table_width = table_width; p.pool_table_width = pool_table_width; p.q_stride = q_stride; p.q_off = q_off;
     p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.pool = pool; p.temp_every = temp_every;
-    p.scale = scale; p.temp_coef = temp_coef;
+    p.scale = scale; p.temp_coef = temp_coef; p.softcap = softcap; p.gate = (const bf16*)gate;
     if (dim <= 32) return prompt_by_value_size<32>(p, n_seqs, max_q_len, stream);
     if (dim <= 64) return prompt_by_value_size<64>(p, n_seqs, max_q_len, stream);
     return prompt_by_value_size<128>(p, n_seqs, max_q_len, stream);

@@ -73,6 +73,18 @@ struct FrVec {
     }
 };
 
+// A gated unit: the gate's activation times up.  kind 1: silu; 2: the tanh form of gelu; 3: both clipped, g = min(gate, limit) and
+// u = clamp(up, -limit, limit), g sigmoid(slope g) (u + 1).
+__device__ __forceinline__ float fr_gated(int kind, float g, float u, float limit, float slope) {
+    if (kind == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    if (kind == 3) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+    }
+    return g / (1.0f + expf(-g)) * u;
+}
+
 // The rotation of one pair of a rotary encoding, the same instructions wherever it is applied.
 __device__ __forceinline__ void fr_rotate(float a, float b, float c, float s, float& ra, float& rb) {
     ra = __fmaf_rn(-b, s, __fmul_rn(a, c));

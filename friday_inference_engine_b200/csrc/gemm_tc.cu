@@ -84,7 +84,8 @@ struct GemmParams {
     int* status;        // 0, or a code when a wait gave up
     int p_rows, q_rows, ldo, out_dtype, bias_dtype, swapped;
     int bn;             // rows of Q per tile: the kernel's BN, or any multiple of 16 below it in the widest instance
-    int act;            // 1, 2: the product's columns are (gate, up) pairs; out gets silu(gate) * up (2: gelu_tanh(gate) * up), half as wide
+    int act;            // 1 to 3: the product's columns are (gate, up) pairs and out, half as wide, gets the gated unit fr_gated(act, ...);
+                        // ACT_RELU_SQUARED: max(x, 0)^2 of every column
     int tiles_p, tiles_q, splits, kb_total, kb_per;
     // Work decomposition.  The first dp_tiles tiles are cut into `splits` equal k ranges each and dealt out round
     // robin (splits = 1: whole tiles).  The remaining sk_tiles tiles ("stream-k"): their k blocks, laid end to end,
@@ -425,6 +426,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
             const float4 b0 = *(const float4*)(s_bias + f0), b1 = *(const float4*)(s_bias + f0 + 4);
             x[0] = a0.x + b0.x; x[1] = a0.y + b0.y; x[2] = a0.z + b0.z; x[3] = a0.w + b0.w;
             x[4] = a1.x + b1.x; x[5] = a1.y + b1.y; x[6] = a1.z + b1.z; x[7] = a1.w + b1.w;
+            if (p.act == ACT_RELU_SQUARED) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const float r = fmaxf(x[j], 0.f);
+                    x[j] = r * r;
+                }
+            }
         };
         auto round8 = [&](const float (&x)[8]) {
             uint4 w;
@@ -441,14 +449,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const float4 a = *(const float4*)(src + 4 * j);
-                x[2 * j] = gated_mul(p.act, a.x, a.y);
-                x[2 * j + 1] = gated_mul(p.act, a.z, a.w);
+                x[2 * j] = gated_mul(p, a.x, a.y);
+                x[2 * j + 1] = gated_mul(p, a.z, a.w);
             }
             __nv_bfloat16* out_at = (__nv_bfloat16*)p.out + (size_t)(q_blk * bn + token) * p.ldo + ((p_blk * TILE_P + f0) >> 1);
             *(uint4*)out_at = round8(x);
         };
         auto finish_rows = [&](int p_blk, int q_blk, int t_lo, int t_cnt) {     // rows t_lo .. t_lo + t_cnt - 1 of the tile
-            if (p.act) {
+            if (p.act && p.act != ACT_RELU_SQUARED) {
                 finish_rows_gated(p_blk, q_blk, t_lo, t_cnt);
                 return;
             }
@@ -1066,9 +1074,10 @@ FR_EXPORT int gemm_tc_fused(const void* x, const void* w, void* out, int out_dty
                             long long scratch_floats, int* counters, int n_counters, int* status, int sm_count,
                             int swap, int bn, int splits, int act, const GemmFusion* fusion, cudaStream_t stream) {
     if (m <= 0 || n <= 0) return FR_OK;
-    if (act < 0 || act > 2) FR_REFUSE("gemm_tc: unknown activation %d", act);
-    if (act && (n % 2 || bias != nullptr || residual != nullptr || out_dtype != FR_BF16))
-        FR_REFUSE("gemm_tc: the gated epilogue needs an even n, bf16 output, no bias and no residual");
+    if (act < 0 || act > ACT_RELU_SQUARED) FR_REFUSE("gemm_tc: unknown activation %d", act);
+    if (act && ((n % 2 && act != ACT_RELU_SQUARED) || bias != nullptr || residual != nullptr || out_dtype != FR_BF16))
+        FR_REFUSE("gemm_tc: an activation in the epilogue needs bf16 output, no bias and no residual, a gated one an even n");
+    if (act == 3 && (fusion == nullptr || !(fusion->act_limit > 0.f))) FR_REFUSE("gemm_tc: the clipped gated unit needs its limit");
     if (k <= 0 || k % 8 || lda % 8 || ldw % 8)
         FR_REFUSE("gemm_tc: k = %d and the row strides (%d, %d) must be multiples of 8 (16-byte rows for TMA)", k, lda, ldw);
     if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) FR_REFUSE("gemm_tc: operands must be 16-byte aligned");

@@ -35,4 +35,6 @@ struct GemmFusion {
     // 6 last accumulator complete, 7 last tile done; of a CTA that sums a tile's partial tiles: 8 it knows, 9 fence
     // passed, 10 partial tiles summed, 11 tile staged, 12 tile written).
     unsigned long long* trace;
+    // (5) Constants of the activation: limit and slope of the clipped gated unit.
+    float act_limit, act_slope;
 };

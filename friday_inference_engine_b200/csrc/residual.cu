@@ -498,8 +498,8 @@ norm_keep_last_kernel(const float* __restrict__ x, FrVec w, float* __restrict__ 
     for (int i = threadIdx.x; i < width; i += blockDim.x) sp[i] = xr[i] * inv * w.at(i);
 }
 
-// out = x + mult * y / sqrt(mean(y^2) + eps) * w; and, if asked for, the norm of `out` that the next sublayer reads:
-// next = out / sqrt(mean(out^2) + eps2) * w2 in the activation dtype
+// out = x + mult * y / sqrt(mean(y^2) + eps) * w; and, if asked for, what the next sublayer reads in the activation dtype:
+// next = out / sqrt(mean(out^2) + eps2) * w2, or out itself (w2 null)
 template <typename TO>
 __global__ void __launch_bounds__(256)
 post_norm_add_kernel(const float* __restrict__ x, const float* __restrict__ y, FrVec w, float eps, float mult, float* __restrict__ out,
@@ -516,9 +516,10 @@ post_norm_add_kernel(const float* __restrict__ x, const float* __restrict__ y, F
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         const float o = fmaf(mult, y[base + i] * inv * w.at(i), x[base + i]);
         out[base + i] = o;
+        if (next != nullptr && w2.p == nullptr) fr_store(next + base + i, o);
         s2 = fmaf(o, o, s2);
     }
-    if (next == nullptr) return;
+    if (next == nullptr || w2.p == nullptr) return;
     s2 = block_sum(s2, partial);
     const float inv2 = 1.0f / sqrtf(s2 / (float)width + eps2);
     for (int i = threadIdx.x; i < width; i += blockDim.x) fr_store(next + base + i, out[base + i] * inv2 * w2.at(i));
@@ -643,10 +644,11 @@ post_norm_add_vec_kernel(const float* __restrict__ x, const float* __restrict__ 
                 s2 = fmaf(o[e], o[e], s2);
             }
             store4(out + base + 4 * i, o);
+            if (next != nullptr && w2.p == nullptr) store4(next + base + 4 * i, o);
             v[k] = make_float4(o[0], o[1], o[2], o[3]);
         }
     }
-    if (next == nullptr) return;
+    if (next == nullptr || w2.p == nullptr) return;
     s2 = block_sum(s2, partial);
     const float inv2 = 1.0f / sqrtf(s2 / (float)width + eps2);
 #pragma unroll
@@ -1077,5 +1079,46 @@ FR_EXPORT int residual_rms_pair_add(const float* x, const float* a, const float*
     if (n_rows <= 0) return FR_OK;
     FR_CUDA(fr_launch(rms_pair_add_kernel, dim3(n_rows), dim3(256), 0, stream, x, a, b, FrVec{wa, w_dtype}, FrVec{wb, w_dtype}, eps, mult, out, width));
     FR_CHECK_LAUNCH("rms_pair_add");
+    return FR_OK;
+}
+
+// ------------------------------------------------------------------ max(z, 0)^2, in place
+namespace {
+template <typename T>
+__global__ void relu_squared_kernel(T* __restrict__ z, long long n, int pieces) {
+    constexpr int PER = 16 / (int)sizeof(T);
+    fr_pdl_wait();
+    fr_pdl_launch();
+    const long long at = (long long)blockIdx.x * blockDim.x + threadIdx.x, step = (long long)gridDim.x * blockDim.x;
+    if (pieces) {
+        for (long long i = at; i < n / PER; i += step) {
+            uint4 raw = ((const uint4*)z)[i];
+            T* e = (T*)&raw;
+#pragma unroll
+            for (int k = 0; k < PER; ++k) {
+                const float v = fmaxf(fr_load(e + k), 0.f);
+                fr_store(e + k, v * v);
+            }
+            ((uint4*)z)[i] = raw;
+        }
+        return;
+    }
+    for (long long i = at; i < n; i += step) {
+        const float v = fmaxf(fr_load(z + i), 0.f);
+        fr_store(z + i, v * v);
+    }
+}
+}  // namespace
+
+FR_EXPORT int residual_relu_squared(void* z, long long n, int dtype, cudaStream_t stream) {
+    if (n <= 0) return FR_OK;
+    const long long per = dtype == FR_F32 ? 4 : 8;
+    const int pieces = n % per == 0 && ((((uintptr_t)z) & 15) == 0);
+    const long long items = pieces ? n / per : n;
+    const int blocks = (int)((items + 255) / 256 < 4096 ? (items + 255) / 256 : 4096);
+    if (dtype == FR_F32) FR_CUDA(fr_launch(relu_squared_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)z, n, pieces));
+    else if (dtype == FR_BF16) FR_CUDA(fr_launch(relu_squared_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (bf16*)z, n, pieces));
+    else FR_REFUSE("relu_squared: unknown dtype %d", dtype);
+    FR_CHECK_LAUNCH("relu_squared");
     return FR_OK;
 }

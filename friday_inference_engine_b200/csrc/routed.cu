@@ -5,7 +5,9 @@
 //                    [rows][experts] that holds each chosen expert's weight and zero elsewhere
 //   scale_by_route   act [rows][experts * inner] *= dense[row][column / inner]: after it, one product over all
 //                    experts' down matrices side by side sums exactly the chosen experts
-//   gate_up          for every (row, choice): act = silu(Wg_e h) * (Wu_e h), expert e's rows read where they lie
+//   route_biased     softmax scores over experts and identity experts (which return their input), a bias for the choice only
+//   shared_and_self  the row's gate times the shared expert's result, plus what its identity experts weigh times the row
+//   gate_up          for every (row, choice): act = silu(Wg_e h) * (Wu_e h) (or the clipped unit), expert e's rows read where they lie
 //   down_combine     out[row] = residual[row] + sum over choices of weight * (Wd_e act)
 //
 // gate_up and down_combine read only the chosen experts' weights, once per (row, choice): the form for one-token
@@ -132,7 +134,7 @@ __global__ void scale_by_route_kernel(T* __restrict__ act, const float* __restri
 template <typename T>
 __global__ void __launch_bounds__(256)
 gate_up_kernel(const T* __restrict__ h, const int* __restrict__ ids, const T* __restrict__ w_gate_up, T* __restrict__ act,
-               int top, int width, int inner, int per_block) {
+               int top, int width, int inner, int per_block, int kind, float limit, float slope) {
     extern __shared__ float hs[];             // [width]
     fr_pdl_wait();
     fr_pdl_launch();
@@ -155,7 +157,7 @@ gate_up_kernel(const T* __restrict__ h, const int* __restrict__ ids, const T* __
         }
         sg = fr_warp_sum(sg);
         su = fr_warp_sum(su);
-        if (lane == 0) fr_store(act + (size_t)pair * inner + f, sg / (1.0f + expf(-sg)) * su);
+        if (lane == 0) fr_store(act + (size_t)pair * inner + f, fr_gated(kind, sg, su, limit, slope));
     }
 }
 
@@ -166,7 +168,7 @@ constexpr int MAX_SHARE = 16;
 template <typename T>
 __global__ void __launch_bounds__(256)
 gate_up_by_expert_kernel(const T* __restrict__ h, const int* __restrict__ ids, const T* __restrict__ w_gate_up, T* __restrict__ act,
-                         int rows, int top, int width, int inner, int per_block) {
+                         int rows, int top, int width, int inner, int per_block, int kind, float limit, float slope) {
     extern __shared__ __align__(16) unsigned char raw[];
     T* hs = (T*)raw;                           // [MAX_SHARE][width]
     __shared__ int pairs[MAX_SHARE];
@@ -240,7 +242,7 @@ gate_up_by_expert_kernel(const T* __restrict__ h, const int* __restrict__ ids, c
         for (int r = 0; r < MAX_SHARE; ++r) {
             if (r < n) {
                 const float a = fr_warp_sum(sg[r]), b = fr_warp_sum(su[r]);
-                if (lane == 0) fr_store(act + (size_t)pairs[r] * inner + f, a / (1.0f + expf(-a)) * b);
+                if (lane == 0) fr_store(act + (size_t)pairs[r] * inner + f, fr_gated(kind, a, b, limit, slope));
             }
         }
     }
@@ -455,9 +457,11 @@ FR_EXPORT int routed_scale_by_route(void* act, const float* dense, int rows, int
     return FR_OK;
 }
 
+// kind, limit, slope: the gated unit (fr_gated)
 FR_EXPORT int routed_gate_up(const void* h, const int* ids, const void* w_gate_up, void* act, int rows, int top, int experts, int width,
-                             int inner, int dtype, cudaStream_t stream) {
+                             int inner, int kind, float limit, float slope, int dtype, cudaStream_t stream) {
     if (rows <= 0) return FR_OK;
+    if (kind < 1 || kind > 3) FR_REFUSE("gate_up: unknown gated unit %d", kind);
     const size_t smem = (size_t)width * sizeof(float);
     if (smem > 200 * 1024) FR_REFUSE("gate_up: width %d does not fit an SM's shared memory", width);
     const int per_block = inner < 64 ? inner : 64;
@@ -472,18 +476,18 @@ FR_EXPORT int routed_gate_up(const void* h, const int* ids, const void* w_gate_u
         const dim3 eg(experts, (inner + eper - 1) / eper);
         if (share > 48 * 1024) FR_CUDA(cudaFuncSetAttribute(gate_up_by_expert_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)share));
         FR_CUDA(fr_launch(gate_up_by_expert_kernel<bf16>, eg, dim3(256), share, stream, (const bf16*)h, ids, (const bf16*)w_gate_up,
-                          (bf16*)act, rows, top, width, inner, eper));
+                          (bf16*)act, rows, top, width, inner, eper, kind, limit, slope));
         FR_CHECK_LAUNCH("gate_up (by expert)");
         return FR_OK;
     }
     if (dtype == FR_F32) {
         if (smem > 48 * 1024) FR_CUDA(cudaFuncSetAttribute(gate_up_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         FR_CUDA(fr_launch(gate_up_kernel<float>, grid, dim3(256), smem, stream, (const float*)h, ids, (const float*)w_gate_up,
-                          (float*)act, top, width, inner, per_block));
+                          (float*)act, top, width, inner, per_block, kind, limit, slope));
     } else if (dtype == FR_BF16) {
         if (smem > 48 * 1024) FR_CUDA(cudaFuncSetAttribute(gate_up_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         FR_CUDA(fr_launch(gate_up_kernel<bf16>, grid, dim3(256), smem, stream, (const bf16*)h, ids, (const bf16*)w_gate_up,
-                          (bf16*)act, top, width, inner, per_block));
+                          (bf16*)act, top, width, inner, per_block, kind, limit, slope));
     } else {
         FR_REFUSE("gate_up: unknown dtype %d", dtype);
     }
@@ -660,5 +664,156 @@ FR_EXPORT int routed_route_scored(const float* logits, int ld, int rows, int exp
     FR_CUDA(fr_launch(route_scored_kernel, dim3((rows + 3) / 4), dim3(128), 0, stream, logits, ld, rows, experts, top,
                       FrVec{bias, bias_dtype}, groups, keep, scale, ids, weights, dense));
     FR_CHECK_LAUNCH("route_scored");
+    return FR_OK;
+}
+
+// ------------------------------------------------------------------ a choice by biased softmax scores, with identity experts
+// Per row: s = softmax of the logits z_0 .. z_(total-1), c_e = s_e + bias_e (bias null: c = s); the `top` of highest c are
+// chosen (the lower index wins a tie), with weights s_e / (the chosen scores' sum + 1e-20).  Experts from `experts` on return
+// their input: their id reads -1 and their weights are added up in self[row] (null: there are none).  fp32; a warp per row.
+namespace {
+
+__global__ void __launch_bounds__(128)
+route_biased_kernel(const float* __restrict__ logits, int ld, int rows, int experts, int total, int top, FrVec bias, int* __restrict__ ids,
+                    float* __restrict__ weights, float* __restrict__ self, float* __restrict__ dense) {
+    fr_pdl_wait();
+    fr_pdl_launch();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int row = blockIdx.x * 4 + warp;
+    if (row >= rows) return;
+    float s[ROUTE_PER_LANE], c[ROUTE_PER_LANE];
+    float big = -INFINITY;
+#pragma unroll
+    for (int i = 0; i < ROUTE_PER_LANE; ++i) {
+        const int e = lane + 32 * i;
+        s[i] = e < total ? logits[(size_t)row * ld + e] : -INFINITY;
+        big = fmaxf(big, s[i]);
+    }
+    big = fr_warp_max(big);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < ROUTE_PER_LANE; ++i) {
+        s[i] = lane + 32 * i < total ? expf(s[i] - big) : 0.f;
+        sum += s[i];
+    }
+    sum = fr_warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < ROUTE_PER_LANE; ++i) {
+        const int e = lane + 32 * i;
+        s[i] /= sum;
+        c[i] = e < total ? s[i] + (bias.p != nullptr ? bias.at(e) : 0.f) : -INFINITY;
+    }
+    if (dense != nullptr)
+        for (int e = lane; e < experts; e += 32) dense[(size_t)row * experts + e] = 0.f;
+    __syncwarp();
+    float my_score = 0.f;                   // lane t keeps the t-th choice
+    int my_id = -1;
+    for (int t = 0; t < top; ++t) {
+        float best = -INFINITY, score = 0.f;
+        int best_e = 0x7fffffff;
+#pragma unroll
+        for (int i = 0; i < ROUTE_PER_LANE; ++i) {
+            const int e = lane + 32 * i;
+            if (e < total && (c[i] > best || (c[i] == best && e < best_e))) {
+                best = c[i];
+                best_e = e;
+                score = s[i];
+            }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, score, o);
+            const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+            if (ob > best || (ob == best && oe < best_e)) {
+                best = ob;
+                best_e = oe;
+                score = os;
+            }
+        }
+        if (best == -INFINITY) best_e = -1;          // no finite score left (a dead row's garbage)
+        if (lane == t) {
+            my_score = best_e >= 0 ? score : 0.f;
+            my_id = best_e;
+        }
+#pragma unroll
+        for (int i = 0; i < ROUTE_PER_LANE; ++i)
+            if (lane + 32 * i == best_e) c[i] = -INFINITY;
+    }
+    const float w = my_score / (fr_warp_sum(my_score) + 1e-20f);
+    const float mine = fr_warp_sum(my_id >= experts ? w : 0.f);
+    if (lane < top) {
+        const bool real = my_id >= 0 && my_id < experts;
+        ids[(size_t)row * top + lane] = real ? my_id : -1;
+        weights[(size_t)row * top + lane] = real ? w : 0.f;
+        if (dense != nullptr && real) dense[(size_t)row * experts + my_id] = w;
+    }
+    if (lane == 0 && self != nullptr) self[row] = mine;
+}
+
+// out = residual + sigmoid(gate[row]) * shared + self[row] * h (each of the three may be absent)
+template <typename T>
+__global__ void __launch_bounds__(256)
+shared_and_self_kernel(const float* __restrict__ residual, const float* __restrict__ shared, const float* __restrict__ gate, int gate_ld,
+                       const float* __restrict__ self, const T* __restrict__ h, float* __restrict__ out, int rows, int width, int by_four) {
+    fr_pdl_wait();
+    fr_pdl_launch();
+    for (int row = blockIdx.y; row < rows; row += gridDim.y) {
+        const size_t base = (size_t)row * width;
+        const float g = gate != nullptr ? 1.0f / (1.0f + expf(-gate[(size_t)row * gate_ld])) : 1.f;
+        const float w = self != nullptr ? self[row] : 0.f;
+        const int step = gridDim.x * blockDim.x, at = blockIdx.x * blockDim.x + threadIdx.x;
+        if (by_four) {
+            for (int c = at * 4; c < width; c += step * 4) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                if (shared != nullptr) {
+                    const float4 s = *(const float4*)(shared + base + c);
+                    v[0] = g * s.x; v[1] = g * s.y; v[2] = g * s.z; v[3] = g * s.w;
+                }
+                if (w != 0.f)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) v[i] = fmaf(w, fr_load(h + base + c + i), v[i]);
+                if (residual != nullptr) {
+                    const float4 r = *(const float4*)(residual + base + c);
+                    v[0] += r.x; v[1] += r.y; v[2] += r.z; v[3] += r.w;
+                }
+                *(float4*)(out + base + c) = make_float4(v[0], v[1], v[2], v[3]);
+            }
+            continue;
+        }
+        for (int c = at; c < width; c += step) {
+            float v = shared != nullptr ? g * shared[base + c] : 0.f;
+            if (w != 0.f) v = fmaf(w, fr_load(h + base + c), v);
+            if (residual != nullptr) v += residual[base + c];
+            out[base + c] = v;
+        }
+    }
+}
+
+}  // namespace
+
+FR_EXPORT int routed_route_biased(const float* logits, int ld, int rows, int experts, int identity, int top, const void* bias, int bias_dtype,
+                                  int* ids, float* weights, float* self, float* dense, cudaStream_t stream) {
+    if (rows <= 0) return FR_OK;
+    const int total = experts + identity;
+    if (experts < 1 || identity < 0 || total > 32 * ROUTE_PER_LANE) FR_REFUSE("route: %d experts and %d that return their input (%d in all)", experts, identity, 32 * ROUTE_PER_LANE);
+    if (top < 1 || top > total || top > 32) FR_REFUSE("route: top %d of %d experts (at most 32)", top, total);
+    if (identity > 0 && self == nullptr) FR_REFUSE("route: experts that return their input need a place for their weights");
+    FR_CUDA(fr_launch(route_biased_kernel, dim3((rows + 3) / 4), dim3(128), 0, stream, logits, ld, rows, experts, total, top,
+                      FrVec{bias, bias_dtype}, ids, weights, self, dense));
+    FR_CHECK_LAUNCH("route_biased");
+    return FR_OK;
+}
+
+// gate: the logits' column that holds the rows' gates, gate_ld apart from row to row
+FR_EXPORT int routed_shared_and_self(const float* residual, const float* shared, const float* gate, int gate_ld, const float* self, const void* h,
+                                     float* out, int rows, int width, int dtype, cudaStream_t stream) {
+    if (rows <= 0 || width <= 0) return FR_OK;
+    const int by_four = width % 4 == 0 && ((((uintptr_t)residual) | ((uintptr_t)shared) | ((uintptr_t)out)) & 15) == 0;
+    const int items = by_four ? width / 4 : width;
+    const dim3 grid((items + 255) / 256, rows < 65535 ? rows : 65535);
+    if (dtype == FR_F32) FR_CUDA(fr_launch(shared_and_self_kernel<float>, grid, dim3(256), 0, stream, residual, shared, gate, gate_ld, self, (const float*)h, out, rows, width, by_four));
+    else if (dtype == FR_BF16) FR_CUDA(fr_launch(shared_and_self_kernel<bf16>, grid, dim3(256), 0, stream, residual, shared, gate, gate_ld, self, (const bf16*)h, out, rows, width, by_four));
+    else FR_REFUSE("shared_and_self: unknown dtype %d", dtype);
+    FR_CHECK_LAUNCH("shared_and_self");
     return FR_OK;
 }

@@ -113,12 +113,10 @@ __device__ __forceinline__ float bias_at(const P& p, int i) {
     return p.bias_dtype == FR_F32 ? ((const float*)p.bias)[i] : __bfloat162float(((const __nv_bfloat16*)p.bias)[i]);
 }
 
-__device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + expf(-g)) * u; }
-// the gate's activation times up: act 1 silu, act 2 the tanh form of gelu
-__device__ __forceinline__ float gated_mul(int act, float g, float u) {
-    if (act == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
-    return silu_mul(g, u);
-}
+// the product's activation: 1 to 3 a gated unit of column pairs (fr_gated), ACT_RELU_SQUARED max(x, 0)^2 of every column
+constexpr int ACT_RELU_SQUARED = 4;
+template <typename P>
+__device__ __forceinline__ float gated_mul(const P& p, float g, float u) { return fr_gated(p.act, g, u, p.f.act_limit, p.f.act_slope); }
 
 // Gated epilogue: rows 2f and 2f+1 of the weight are gate f and up f.  Must be called by whole warps.
 template <typename P>
@@ -128,7 +126,7 @@ __device__ __forceinline__ void finish16_gated(const P& p, int gi, int gj0, floa
         if (gi >= p.p_rows) return;
         float r[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) r[j] = gated_mul(p.act, v[2 * j], v[2 * j + 1]);
+        for (int j = 0; j < 8; ++j) r[j] = gated_mul(p, v[2 * j], v[2 * j + 1]);
         const int oj0 = gj0 >> 1, o_cols = p.q_rows >> 1;
         __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)gi * p.ldo + oj0;
         if (oj0 + 8 <= o_cols && (p.ldo % 8 == 0) && (((uintptr_t)p.out & 15) == 0)) {
@@ -147,14 +145,22 @@ __device__ __forceinline__ void finish16_gated(const P& p, int gi, int gj0, floa
         for (int j = 0; j < 16; ++j) up[j] = __shfl_xor_sync(0xffffffffu, v[j], 1);
         if ((gi & 1) || gi >= p.p_rows) return;
         for (int j = 0; j < 16 && gj0 + j < p.q_rows; ++j)
-            ((__nv_bfloat16*)p.out)[(size_t)(gj0 + j) * p.ldo + (gi >> 1)] = __float2bfloat16_rn(gated_mul(p.act, v[j], up[j]));
+            ((__nv_bfloat16*)p.out)[(size_t)(gj0 + j) * p.ldo + (gi >> 1)] = __float2bfloat16_rn(gated_mul(p, v[j], up[j]));
     }
 }
 
 // Bias, residual, rounding and store of 16 consecutive q-columns of P-row gi.
 template <typename P>
 __device__ __forceinline__ void finish16(const P& p, int gi, int gj0, float (&v)[16]) {
-    if (p.act) return finish16_gated(p, gi, gj0, v);
+    if (p.act == ACT_RELU_SQUARED) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+            const float x = fmaxf(v[j], 0.f);
+            v[j] = x * x;
+        }
+    } else if (p.act) {
+        return finish16_gated(p, gi, gj0, v);
+    }
     if (gi >= p.p_rows) return;
     if (!p.swapped) {
         // out[gi][gj0 .. gj0+15]

@@ -105,8 +105,9 @@ public:
     Tensor embedding(const int* tokens, int64_t n, const Tensor& table, Tensor* out = nullptr);
     Tensor gather_rows(const int* rows, int64_t n, const Tensor& src);
     Tensor rmsnorm(const Tensor& x, const Tensor& weight, float eps, Tensor* out = nullptr);
-    // columns alternate gate, up; act 1: silu(gate) * up, act 2: gelu_tanh(gate) * up
-    Tensor swiglu(const Tensor& gate_up, int act = 1);
+    // columns alternate gate, up; act 1: silu(gate) * up, act 2: gelu_tanh(gate) * up, act 3 (with a limit L and a slope a):
+    // g sigmoid(a g) (u + 1) with g = min(gate, L), u = clamp(up, -L, L)
+    Tensor swiglu(const Tensor& gate_up, int act = 1, float limit = 0.f, float slope = 1.f);
     // Rotates q and k inside qkv [rows, (nq + 2 nkv) * hd] (denominators null: no rotation) and, if the view
     // may be written, stores k and v in the cache rows of (row_seq, row_pos).
     void rope_kv_write(Tensor& qkv, const int* row_seq, const int* row_pos, const float* denominators, int rotary_dim,
@@ -119,6 +120,7 @@ public:
     // y = x / sqrt(mean(x^2) + eps) * (offset + weight), x and y in dtypes of their own
     Tensor rmsnorm_to(const Tensor& x, const Tensor& weight, float offset, float eps, DType out_dtype);
     Tensor concat_cast(const Tensor& a, const Tensor& b, DType out_dtype);            // [a, b] side by side
+    Tensor cast_rows(const Tensor& x, DType out_dtype);                               // x itself if it has that dtype
     // residual (fp32) + alpha * y (+ beta * z): a new fp32 tensor, or `residual` itself with in_place
     Tensor add_scaled(const Tensor& residual, const Tensor& y, float alpha, const Tensor* z = nullptr, float beta = 0.f,
                       bool in_place = false);
@@ -136,12 +138,13 @@ public:
     // the width per sequence), which then keeps the h of the step's last row
     Tensor norm_shift(const Tensor& x, const Tensor& weight, float eps, const Tensor& shift, const CacheView& view, const StepContext& ctx,
                       DType out_dtype);
-    // x + mult * y / sqrt(mean(y^2) + eps) * weight (x, y 32-bit); with next_weight also the norm of that sum in `next_dtype`
-    // (what the sublayer after it reads), returned through `next`
+    // x + mult * y / sqrt(mean(y^2) + eps) * weight (x, y 32-bit); with `next` also what the sublayer after it reads, in
+    // `next_dtype`: the norm of that sum with next_weight, or (next_weight null) the sum itself
     Tensor post_norm_add(const Tensor& x, const Tensor& y, const Tensor& weight, float eps, float mult, const Tensor* next_weight = nullptr,
                          float next_eps = 0.f, DType next_dtype = DType::F32, Tensor* next = nullptr);
     // in place: z > 0: softplus(p) z^2 + z / 2; z <= 0: (1/2 + softplus(q)) (e^z - 1 - z) + z / 2; pq = (p, q)
     void two_sided_act(Tensor& z, const Tensor& pq);
+    void relu_squared(Tensor& z);                             // in place: max(z, 0)^2
     // keys [n_kv_heads][head_dim] at column k_off and values [n_kv_heads][v_head_dim] at column v_off of every row of
     // `src` go to the cache rows of (row_seq, row_pos)
     void kv_store(const Tensor& src, int64_t k_off, int64_t v_off, const CacheView& view, const StepContext& ctx);
@@ -176,6 +179,17 @@ public:
         const Tensor* bonus = nullptr;  // [heads * dk]: read the state before the update, with bonus * k v^T for the present token
         const Tensor* carry = nullptr;  // rows whose last one per sequence is kept at the start of the state
     };
+    // S <- decay_h S + k v^T, o = S^T q with a constant decay per head (device table [heads]) and q, k, v = silu of the columns of
+    // `proj` at the given offsets (rounded to its dtype); the state starts at state_offset of a sequence's tensor.
+    // -> [rows, heads * dv] fp32.  Prompts in bfloat16 run in chunks of tokens on the tensor cores, their states in 32-bit.
+    struct DecaySpec {
+        int heads = 0, dk = 0, dv = 0;
+        const float* decay = nullptr;
+        int64_t q_off = 0, k_off = 0, v_off = 0;
+    };
+    Tensor decay_scan(const Tensor& proj, const DecaySpec& spec, const CacheView& view, const StepContext& ctx);
+    // o [rows, n] fp32 -> o / sqrt(mean(o^2) + eps) * weight * sigmoid(gate) in `dtype`: one norm over the whole row
+    Tensor row_norm_gate(const Tensor& o, const Tensor& gate, const Tensor& weight, float eps, DType dtype);
     // q, k [rows, >= heads * dk], v [rows, >= heads * dv] (the tensors' row strides are used), z [rows, heads * dk] fp32
     Tensor state_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& z, const ScanSpec& spec, const CacheView& view,
                       const StepContext& ctx);
@@ -222,11 +236,16 @@ public:
         const Tensor* sink = nullptr;   // [heads]: exp(sink_h) joins head h's denominator
         const Tensor* q_norm = nullptr; // [dim]: RMS norm of every query head with this weight (null: none)
         const Tensor* k_norm = nullptr;
+        bool norm_whole = false;        // one RMS norm over all query heads at once with a weight [heads * dim], likewise the keys
         float eps = 1e-5f;
         const float* freq = nullptr;    // device [rot / 2]: pairs (i, i + rot / 2) of q and k turn by pos * freq[i]; null: no rotation
+        bool neighbours = false;        // the pairs are (2i, 2i + 1) instead
         float rot_mult = 1.f;
         int rot = 0;
-        int64_t q_off = 0, k_off = 0, v_off = -1;       // columns of the stacked projection; v_off < 0: the values are the keys
+        float softcap = 0.f;            // > 0: score <- cap * tanh(score / cap)
+        // columns of the stacked projection; v_off < 0: the values are the keys; k_off < 0: queries only (another layer's keys and values)
+        int64_t q_off = 0, k_off = 0, v_off = -1;
+        int64_t gate_off = -1;          // >= 0: head h's result is multiplied by sigmoid of column gate_off + h
     };
     // q (normed, rotated) goes back into proj; k (normed, rotated) and v go to the cache rows of the step's tokens; with
     // pooled blocks the blocks' sums (`pooled`: a view of 32-bit rows, one per `pool` positions) take the step's tokens
@@ -263,20 +282,28 @@ public:
     // ---- routed experts (csrc/routed.cu)
     struct Routing {
         Tensor ids, weights, dense;     // [rows, top] int32, [rows, top] fp32, [rows, experts] fp32 (if asked for)
+        Tensor self;                    // [rows] fp32: what the chosen identity experts weigh together (undefined: there are none)
     };
     Routing route(const Tensor& logits, int top, bool softmax_all, bool with_dense);
     // scores sigmoid(logit); the choice runs on score + bias (null: none) among the experts of the `keep` best of `groups`
     // equally sized runs of adjacent experts (a group counts as the sum of its two largest); weights = score * scale of the chosen
     Routing route_scored(const Tensor& logits, int top, const Tensor* bias, int groups, int keep, float scale, bool with_dense);
+    // scores softmax over the first `experts` + `identity` columns of the logits; the choice runs on score + bias (null: none); weights =
+    // the chosen scores divided by their sum + 1e-20.  A chosen identity expert (the last `identity` of them) has id -1 and adds its
+    // weight to `self`.
+    Routing route_biased(const Tensor& logits, int experts, int identity, int top, const Tensor* bias, bool with_dense);
+    // residual (null: none) + sigmoid(gate column of the logits) * shared (null: none) + self * h, 32-bit rows
+    Tensor shared_and_self(const Tensor* residual, const Tensor* shared, const Tensor* logits, int64_t gate_col, const Tensor* self, const Tensor& h);
     void scale_by_route(Tensor& act, const Tensor& dense, int experts, int inner);
-    Tensor expert_gate_up(const Tensor& h, const Routing& r, const Tensor& w_gate_up, int top, int inner);
+    Tensor expert_gate_up(const Tensor& h, const Routing& r, const Tensor& w_gate_up, int top, int inner, int act = 1, float limit = 0.f,
+                          float slope = 1.f);
     Tensor expert_down_combine(const Tensor& act, const Routing& r, const Tensor& w_down, const Tensor& residual, int top, int inner);
     // Many rows: the rows are gathered expert by expert and every expert with rows runs its two products on the tensor
     // cores over its own rows only.  The host reads the experts' row counts (one small copy and a wait per call), so this
     // is for prompts, never inside a captured step.  w_gate_up [experts * 2 * inner, width] (gate and up row by row in
     // turn), w_down [width, experts * inner].
     Tensor experts_grouped(const Tensor& h, const Routing& r, const Tensor& w_gate_up, const Tensor& w_down, const Tensor& residual,
-                           int top, int inner);
+                           int top, int inner, int act = 1, float limit = 0.f, float slope = 1.f);
 
     // ---- matrix products: x [rows, k] @ weight [n, k]^T (+ bias [n]) (+ residual [rows, n])
     Tensor linear(const Rows& x, const Tensor& weight, const Tensor* bias = nullptr, const Tensor* residual = nullptr,
@@ -291,8 +318,10 @@ public:
                           const int* row_pos, const float* denominators, int rotary_dim, int n_heads, int n_kv_heads,
                           int head_dim, const CacheView* view);
     // silu(x Wg^T) * (x Wu^T) for weight_pairs [2 * inner, k] whose rows alternate gate, up.
-    // act 2: the tanh form of gelu instead of silu
-    Tensor linear_swiglu(const Rows& x, const Tensor& weight_pairs, int act = 1);
+    // act 2, 3: the other kinds of swiglu()
+    Tensor linear_swiglu(const Rows& x, const Tensor& weight_pairs, int act = 1, float limit = 0.f, float slope = 1.f);
+    // max(x W^T, 0)^2, in the product's epilogue where the tensor cores run it
+    Tensor linear_relu_squared(const Rows& x, const Tensor& weight);
     Tensor materialize(const Rows& h);
 
     // ---- attention of the step's rows over the paged cache.  q: the buffer that holds the queries, row stride

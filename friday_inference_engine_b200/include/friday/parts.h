@@ -269,6 +269,9 @@ public:
     // A layer norm (x - mean) / sqrt(variance + eps) * weight + bias answers with its parts (bias undefined: none), so that
     // a block may run it inside a kernel that does more (a short convolution after it).
     virtual bool layer_parts(Tensor* weight, Tensor* bias, float* eps) const { return false; }
+    // True for the part that leaves rows as they are (in the activation dtype): a block whose sublayers read the stream itself
+    // names it where another block has a norm, and a kernel that would run the norm only rounds instead.
+    virtual bool identity() const { return false; }
 };
 
 class Position : public Part {

@@ -109,7 +109,8 @@ FAMILY(Residual, residual, "residual", resolve(h, fam, "residual_norm_cast", t.n
        resolve(h, fam, "residual_embed_pos", t.embed_pos); resolve(h, fam, "residual_norm_shift", t.norm_shift);
        resolve(h, fam, "residual_post_norm_add", t.post_norm_add); resolve(h, fam, "residual_two_sided_act", t.two_sided_act);
        resolve(h, fam, "residual_embed_pair", t.embed_pair); resolve(h, fam, "residual_norm_conv", t.norm_conv);
-       resolve(h, fam, "residual_norm_conv_state", t.norm_conv_state); resolve(h, fam, "residual_rms_pair_add", t.rms_pair_add);)
+       resolve(h, fam, "residual_norm_conv_state", t.norm_conv_state); resolve(h, fam, "residual_rms_pair_add", t.rms_pair_add);
+       resolve(h, fam, "residual_relu_squared", t.relu_squared);)
 FAMILY(Recurrence, recurrence, "recurrence", resolve(h, fam, "recurrence_shift_mix", t.shift_mix);
        resolve(h, fam, "recurrence_tanh_rows", t.tanh_rows); resolve(h, fam, "recurrence_scan", t.scan);
        resolve(h, fam, "recurrence_scan_plan", t.scan_plan);
@@ -119,11 +120,14 @@ FAMILY(Routed, routed, "routed", resolve(h, fam, "routed_route", t.route);
        resolve(h, fam, "routed_down_combine", t.down_combine);
        resolve(h, fam, "routed_down_scratch_floats", t.down_scratch_floats);
        resolve(h, fam, "routed_sort_pairs", t.sort_pairs); resolve(h, fam, "routed_combine", t.combine);
-       resolve(h, fam, "routed_route_scored", t.route_scored);)
+       resolve(h, fam, "routed_route_scored", t.route_scored); resolve(h, fam, "routed_route_biased", t.route_biased);
+       resolve(h, fam, "routed_shared_and_self", t.shared_and_self);)
 FAMILY(AttentionTalk, attention_talk, "attention_talk", resolve(h, fam, "attention_talk_store", t.store);
        resolve(h, fam, "attention_talk_scratch_floats", t.scratch_floats); resolve(h, fam, "attention_talk_rows", t.rows);
        resolve(h, fam, "attention_talk_prompt_scratch_floats", t.prompt_scratch_floats);
        resolve(h, fam, "attention_talk_prompt", t.prompt);)
+FAMILY(LinearDecay, linear_decay, "linear_decay", resolve(h, fam, "linear_decay_scratch_floats", t.scratch_floats);
+       resolve(h, fam, "linear_decay_run", t.run); resolve(h, fam, "linear_decay_row_norm_gate", t.row_norm_gate);)
 FAMILY(Delta, delta, "delta", resolve(h, fam, "delta_conv_prepare", t.conv_prepare);
        resolve(h, fam, "delta_conv_state", t.conv_state); resolve(h, fam, "delta_scan", t.scan);
        resolve(h, fam, "delta_general_prepare", t.general_prepare); resolve(h, fam, "delta_general_scan", t.general_scan);)

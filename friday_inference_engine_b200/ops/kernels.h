@@ -23,7 +23,7 @@ struct Rowwise {
     int (*gather_rows)(const int*, const void*, void*, int, int, int, cudaStream_t);
     int (*rmsnorm)(const void*, const void*, int, void*, int, int, float, int, cudaStream_t);
     int (*swiglu)(const void*, void*, int, int, int, cudaStream_t);
-    int (*gated_act)(const void*, void*, int, int, int, int, cudaStream_t);
+    int (*gated_act)(const void*, void*, int, int, int, float, float, int, cudaStream_t);
     int (*rope_kv_write)(void*, const int*, const int*, const float*, int, int, int, int, void*, void*, const int*, int, int,
                          int, int, int, cudaStream_t);
     int (*advance)(int*, const int*, int*, int*, const int*, int*, int, cudaStream_t);
@@ -81,6 +81,7 @@ struct Residual {
     int (*norm_conv_state)(const float*, const void*, const void*, int, int, int, float*, long long, long long, const int*, const int*,
                            const int*, int, int, float, cudaStream_t);
     int (*rms_pair_add)(const float*, const float*, const float*, const void*, const void*, int, float, float, float*, int, int, cudaStream_t);
+    int (*relu_squared)(void*, long long, int, cudaStream_t);
 };
 struct Recurrence {
     last_error_fn last_error;
@@ -93,6 +94,13 @@ struct Recurrence {
     int (*scan_plan)(int, int, int, int, int, long long*);
     int (*head_norm_gate)(const float*, const void*, int, void*, const void*, int, int, const int*, int, int, int, float, float, int,
                           int, cudaStream_t);
+};
+struct LinearDecay {
+    last_error_fn last_error;
+    long long (*scratch_floats)(int, int, int, int, int, int);
+    int (*run)(const void*, int, int, int, int, const float*, float*, float*, long long, const int*, const int*, const int*, const int*, int, int,
+               int, int, int, float*, int, cudaStream_t);
+    int (*row_norm_gate)(const float*, const void*, int, void*, const void*, int, int, int, float, int, cudaStream_t);
 };
 struct Delta {
     last_error_fn last_error;
@@ -109,18 +117,18 @@ struct Delta {
 };
 struct AttentionPooled {
     last_error_fn last_error;
-    int (*prepare)(void*, int, int, int, int, const void*, const void*, int, float, const float*, float, int, void*, void*, const int*, int,
-                   int, const int*, const int*, int, int, int, int, int, int, int, cudaStream_t);
+    int (*prepare)(void*, int, int, int, int, const void*, const void*, int, float, const float*, float, int, int, int, void*, void*, const int*,
+                   int, int, const int*, const int*, int, int, int, int, int, int, int, cudaStream_t);
     int (*pool)(const void*, const void*, float*, float*, const int*, int, const int*, int, int, const int*, const int*, int, int, int, int,
                 int, int, int, cudaStream_t);
     long long (*scratch_floats)(int, int, int, int);
     int (*rows)(const void*, int, int, void*, const void*, const void*, const float*, const float*, const int*, int, const int*, int, int,
-                const int*, const int*, int, int, int, int, int, int, int, float, float, int, const void*, int, int, float*, int,
-                cudaStream_t);
+                const int*, const int*, int, int, int, int, int, int, int, float, float, int, float, const void*, int, const void*, int, float*,
+                int, cudaStream_t);
     int (*prompt_fits)(int, int, int);
     int (*prompt)(const void*, int, int, void*, const void*, const void*, const float*, const float*, const int*, int, const int*, int, int,
-                  const int*, const int*, const int*, int, int, int, int, int, int, int, int, float, float, int, const void*, int,
-                  cudaStream_t);
+                  const int*, const int*, const int*, int, int, int, int, int, int, int, int, float, float, int, float, const void*, int,
+                  const void*, cudaStream_t);
 };
 struct AttentionLatent {
     last_error_fn last_error;
@@ -140,13 +148,15 @@ struct Routed {
     last_error_fn last_error;
     int (*route)(const float*, int, int, int, int, int, int*, float*, float*, cudaStream_t);
     int (*scale_by_route)(void*, const float*, int, int, int, int, cudaStream_t);
-    int (*gate_up)(const void*, const int*, const void*, void*, int, int, int, int, int, int, cudaStream_t);
+    int (*gate_up)(const void*, const int*, const void*, void*, int, int, int, int, int, int, float, float, int, cudaStream_t);
     int (*down_combine)(const void*, const int*, const float*, const void*, int, const void*, void*, int, int, int, int, int, int,
                         float*, int, cudaStream_t);
     long long (*down_scratch_floats)(int, int, int, int, int);
     int (*sort_pairs)(const int*, int, int, int, int*, int*, int*, cudaStream_t);
     int (*combine)(const float*, const int*, const float*, const int*, const void*, void*, int, int, int, int, cudaStream_t);
     int (*route_scored)(const float*, int, int, int, int, const void*, int, int, int, float, int*, float*, float*, cudaStream_t);
+    int (*route_biased)(const float*, int, int, int, int, int, const void*, int, int*, float*, float*, float*, cudaStream_t);
+    int (*shared_and_self)(const float*, const float*, const float*, int, const float*, const void*, float*, int, int, int, cudaStream_t);
 };
 struct AttentionTalk {
     last_error_fn last_error;
@@ -188,6 +198,7 @@ const AttentionWindow& attention_window();
 const Residual& residual();
 const Recurrence& recurrence();
 const Routed& routed();
+const LinearDecay& linear_decay();
 const Delta& delta();
 const AttentionLatent& attention_latent();
 const AttentionTalk& attention_talk();

@@ -139,13 +139,13 @@ Tensor Ops::rmsnorm(const Tensor& x, const Tensor& weight, float eps, Tensor* ou
     return o;
 }
 
-Tensor Ops::swiglu(const Tensor& gate_up, int act) {
+Tensor Ops::swiglu(const Tensor& gate_up, int act, float limit, float slope) {
     if (!gate_up.contiguous() || gate_up.cols() % 2) throw KernelError("swiglu: rows must be contiguous pairs (gate, up)");
     const int64_t inner = gate_up.cols() / 2;
     Tensor o = alloc(gate_up.dtype, gate_up.rows(), inner);
     const auto& k = kernels::rowwise();
     Timed t(*this, Other);
-    call(launches_, k, k.gated_act(gate_up.data, o.data, (int)gate_up.rows(), (int)inner, act, code(gate_up.dtype), stream_), "gated_act");
+    call(launches_, k, k.gated_act(gate_up.data, o.data, (int)gate_up.rows(), (int)inner, act, limit, slope, code(gate_up.dtype), stream_), "gated_act");
     return o;
 }
 
@@ -211,6 +211,16 @@ Tensor Ops::concat_cast(const Tensor& a, const Tensor& b, DType out_dtype) {
     Timed t(*this, Other);
     call(launches_, k, k.concat_cast(a.data, b.data, code(a.dtype), o.data, code(out_dtype), (int)a.rows(), (int)a.cols(),
                                      (int)b.cols(), stream_), "concat_cast");
+    return o;
+}
+
+Tensor Ops::cast_rows(const Tensor& x, DType out_dtype) {
+    if (x.dtype == out_dtype) return x;
+    if (!x.contiguous()) throw KernelError("cast_rows: rows must be contiguous");
+    Tensor o = alloc(out_dtype, x.rows(), x.cols());
+    const auto& k = kernels::residual();
+    Timed t(*this, Other);
+    call(launches_, k, k.concat_cast(x.data, x.data, code(x.dtype), o.data, code(out_dtype), (int)x.rows(), (int)x.cols(), 0, stream_), "concat_cast");
     return o;
 }
 
@@ -291,12 +301,12 @@ Tensor Ops::post_norm_add(const Tensor& x, const Tensor& y, const Tensor& weight
         weight.numel() != x.cols() || (next_weight && (!next || next_weight->numel() != x.cols())))
         throw KernelError("post_norm_add: a contiguous 32-bit stream, a 32-bit addend of its size and weights of its width");
     Tensor o = alloc(DType::F32, x.rows(), x.cols());
-    if (next_weight) *next = alloc(next_dtype, x.rows(), x.cols());
+    if (next) *next = alloc(next_dtype, x.rows(), x.cols());
     const auto& k = kernels::residual();
     Timed t(*this, Other);
     call(launches_, k, k.post_norm_add((const float*)x.data, (const float*)y.data, weight.data, code(weight.dtype), eps, mult,
                                        (float*)o.data, next_weight ? next_weight->data : nullptr, next_weight ? code(next_weight->dtype) : 0,
-                                       next_eps, next_weight ? next->data : nullptr, code(next_dtype), (int)x.rows(), (int)x.cols(), stream_),
+                                       next_eps, next ? next->data : nullptr, code(next_dtype), (int)x.rows(), (int)x.cols(), stream_),
          "post_norm_add");
     return o;
 }
@@ -306,6 +316,13 @@ void Ops::two_sided_act(Tensor& z, const Tensor& pq) {
     const auto& k = kernels::residual();
     Timed t(*this, Other);
     call(launches_, k, k.two_sided_act(z.data, (long long)z.numel(), code(z.dtype), pq.data, code(pq.dtype), stream_), "two_sided_act");
+}
+
+void Ops::relu_squared(Tensor& z) {
+    if (!z.contiguous()) throw KernelError("relu_squared: rows must be contiguous");
+    const auto& k = kernels::residual();
+    Timed t(*this, Other);
+    call(launches_, k, k.relu_squared(z.data, (long long)z.numel(), code(z.dtype), stream_), "relu_squared");
 }
 
 // ------------------------------------------------------------------ attention whose heads talk before the softmax
@@ -521,11 +538,14 @@ static void check_pooled(const Ops::PooledSpec& s, const CacheView& tokens, cons
 void Ops::pooled_store(Tensor& proj, const PooledSpec& s, const CacheView& tokens, const CacheView* pooled, const StepContext& ctx) {
     check_pooled(s, tokens, pooled, proj.dtype);
     const auto& k = kernels::attention_pooled();
+    if ((s.k_off < 0) == tokens.write) throw KernelError("pooled attention: a layer that reads another's keys and values does not write them, every other one does");
+    if (s.norm_whole && ((s.q_norm && s.q_norm->numel() != (int64_t)s.heads * s.dim) || (s.k_norm && s.k_norm->numel() != (int64_t)s.kv_heads * s.dim)))
+        throw KernelError("pooled attention: a norm over all heads has a weight per channel of every head");
     const int ndt = s.q_norm ? code(s.q_norm->dtype) : 0;
     if (s.q_norm && s.k_norm && s.q_norm->dtype != s.k_norm->dtype) throw KernelError("pooled attention: the two norm weights have one dtype");
     Timed t(*this, Other);
-    call(launches_, k, k.prepare(proj.data, (int)proj.ld, (int)s.q_off, (int)s.k_off, (int)(s.v_off < 0 ? 0 : s.v_off), s.q_norm ? s.q_norm->data : nullptr,
-                                 s.k_norm ? s.k_norm->data : nullptr, ndt, s.eps, s.freq, s.rot_mult, s.rot, tokens.k_pool,
+    call(launches_, k, k.prepare(proj.data, (int)proj.ld, (int)s.q_off, (int)(s.k_off < 0 ? 0 : s.k_off), (int)(s.v_off < 0 ? 0 : s.v_off), s.q_norm ? s.q_norm->data : nullptr,
+                                 s.k_norm ? s.k_norm->data : nullptr, ndt, s.eps, s.freq, s.rot_mult, s.rot, s.neighbours ? 1 : 0, s.norm_whole ? 1 : 0, tokens.k_pool,
                                  s.v_off < 0 ? nullptr : tokens.v_pool, tokens.block_table, tokens.table_width, tokens.page_size, ctx.row_seq,
                                  ctx.row_pos, (int)proj.rows(), s.heads, s.kv_heads, s.dim, s.vdim, tokens.write ? 1 : 0, code(proj.dtype), stream_),
          "pooled prepare");
@@ -539,6 +559,7 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
     check_pooled(s, tokens, pooled, proj.dtype);
     const auto& k = kernels::attention_pooled();
     Tensor out = alloc(proj.dtype, proj.rows(), (int64_t)s.heads * s.vdim);
+    const void* gate = s.gate_off >= 0 ? (const char*)proj.data + (size_t)s.gate_off * dtype_size(proj.dtype) : nullptr;
     const float* pk = pooled ? (const float*)pooled->k_pool : nullptr;
     const float* pv = pooled ? (const float*)pooled->v_pool : nullptr;
     const int* ptable = pooled ? pooled->block_table : nullptr;
@@ -549,8 +570,8 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
     if (tc) {
         call(launches_, k, k.prompt(proj.data, (int)proj.ld, (int)s.q_off, out.data, tokens.k_pool, tokens.v_pool, pk, pv, tokens.block_table,
                                     tokens.table_width, ptable, pwidth, tokens.page_size, ctx.seq_start, ctx.seq_qlen, ctx.seq_pos0, ctx.n_seqs,
-                                    ctx.max_q_len, s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.pool, s.scale, s.temp_coef, s.temp_every,
-                                    s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, stream_), "pooled prompt");
+                                    ctx.max_q_len, s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.pool, s.scale, s.temp_coef, s.temp_every, s.softcap,
+                                    s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, stream_), "pooled prompt");
         return out;
     }
     // keys that a row can face: its window (or everything before it) and the pooled blocks
@@ -560,8 +581,8 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
     float* scratch = scratch_floats(k.scratch_floats((int)proj.rows(), s.heads, s.vdim, splits));
     call(launches_, k, k.rows(proj.data, (int)proj.ld, (int)s.q_off, out.data, tokens.k_pool, tokens.v_pool, pk, pv, tokens.block_table,
                               tokens.table_width, ptable, pwidth, tokens.page_size, ctx.row_seq, ctx.row_pos, (int)proj.rows(), s.heads, s.kv_heads,
-                              s.dim, s.vdim, s.window, s.pool, s.scale, s.temp_coef, s.temp_every, s.sink ? s.sink->data : nullptr,
-                              s.sink ? code(s.sink->dtype) : 0, splits, scratch, code(proj.dtype), stream_), "pooled rows");
+                              s.dim, s.vdim, s.window, s.pool, s.scale, s.temp_coef, s.temp_every, s.softcap, s.sink ? s.sink->data : nullptr,
+                              s.sink ? code(s.sink->dtype) : 0, gate, splits, scratch, code(proj.dtype), stream_), "pooled rows");
     ++launches_;                                     // the merge
     return out;
 }
@@ -627,6 +648,34 @@ Tensor Ops::head_norm_gate(const Tensor& o, const Tensor& gate, const Tensor& we
     call(launches_, k, k.head_norm_gate((const float*)o.data, gate.data, (int)gate.ld, out.data, weight.data, code(weight.dtype),
                                         weight_per_head ? 1 : 0, ctx.row_seq, (int)o.rows(), heads, dv, eps, out_scale,
                                         gate_sigmoid ? 1 : 0, code(dtype), stream_), "head_norm_gate");
+    return out;
+}
+
+Tensor Ops::decay_scan(const Tensor& proj, const DecaySpec& s, const CacheView& view, const StepContext& ctx) {
+    if (view.kind != CacheRequest::State || !view.state.defined() || view.state.dtype != DType::F32) throw KernelError("decay_scan needs a 32-bit state view");
+    const long long stride = view.state.numel() / view.state.shape[0];
+    if ((long long)s.heads * s.dk * s.dv > stride) throw KernelError("decay_scan: the state is smaller than the heads' matrices");
+    Tensor out = alloc(DType::F32, proj.rows(), (int64_t)s.heads * s.dv);
+    const auto& k = kernels::linear_decay();
+    // FRIDAY_DECAY_CHUNKS=0 keeps prompts on the token-by-token kernel (for comparisons)
+    const long long need = !ctx.decode && env_on("FRIDAY_DECAY_CHUNKS") ? k.scratch_floats(ctx.n_seqs, ctx.max_q_len, s.heads, s.dk, s.dv, code(proj.dtype)) : 0;
+    float* scratch = need > 0 ? scratch_floats(need) : nullptr;
+    Timed t(*this, Attention);
+    call(launches_, k, k.run(proj.data, (int)proj.ld, (int)s.q_off, (int)s.k_off, (int)s.v_off, s.decay, (float*)out.data, (float*)view.state.data, stride,
+                             ctx.row_seq, ctx.seq_start, ctx.seq_qlen, view.seq_slots, ctx.n_seqs, ctx.max_q_len, s.heads, s.dk, s.dv, scratch,
+                             code(proj.dtype), stream_), "linear_decay");
+    if (scratch) launches_ += 2;
+    return out;
+}
+
+Tensor Ops::row_norm_gate(const Tensor& o, const Tensor& gate, const Tensor& weight, float eps, DType dtype) {
+    if (o.dtype != DType::F32 || !o.contiguous() || gate.dtype != dtype || gate.cols() != o.cols() || gate.rows() != o.rows() || weight.numel() != o.cols())
+        throw KernelError("row_norm_gate: fp32 rows, a gate of their size in the result's dtype, a weight per channel");
+    Tensor out = alloc(dtype, o.rows(), o.cols());
+    const auto& k = kernels::linear_decay();
+    Timed t(*this, Other);
+    call(launches_, k, k.row_norm_gate((const float*)o.data, gate.data, (int)gate.ld, out.data, weight.data, code(weight.dtype), (int)o.rows(), (int)o.cols(),
+                                       eps, code(dtype), stream_), "row_norm_gate");
     return out;
 }
 
@@ -811,6 +860,37 @@ Ops::Routing Ops::route_scored(const Tensor& logits, int top, const Tensor* bias
     return r;
 }
 
+Ops::Routing Ops::route_biased(const Tensor& logits, int experts, int identity, int top, const Tensor* bias, bool with_dense) {
+    if (logits.dtype != DType::F32 || logits.cols() < experts + identity) throw KernelError("route: router logits are float32, one per expert");
+    if (bias && bias->numel() != experts + identity) throw KernelError("route: the choice bias has a number per expert");
+    Routing r;
+    const int64_t rows = logits.rows();
+    r.ids = Tensor::make(arena->alloc((size_t)rows * top * sizeof(int)), DType::I32, {rows, (int64_t)top});
+    r.weights = alloc(DType::F32, rows, top);
+    if (identity > 0) r.self = alloc(DType::F32, rows, 1);
+    if (with_dense) r.dense = alloc(DType::F32, rows, experts);
+    const auto& k = kernels::routed();
+    Timed t(*this, Other);
+    call(launches_, k, k.route_biased((const float*)logits.data, (int)logits.ld, (int)rows, experts, identity, top, bias ? bias->data : nullptr,
+                                      bias ? code(bias->dtype) : 0, (int*)r.ids.data, (float*)r.weights.data,
+                                      identity > 0 ? (float*)r.self.data : nullptr, with_dense ? (float*)r.dense.data : nullptr, stream_), "route_biased");
+    return r;
+}
+
+Tensor Ops::shared_and_self(const Tensor* residual, const Tensor* shared, const Tensor* logits, int64_t gate_col, const Tensor* self, const Tensor& h) {
+    for (const Tensor* t : {residual, shared})
+        if (t && (t->dtype != DType::F32 || !t->contiguous() || t->numel() != h.numel())) throw KernelError("shared_and_self: contiguous 32-bit rows of the input's size");
+    if (!h.contiguous() || (logits && (logits->dtype != DType::F32 || gate_col >= logits->cols()))) throw KernelError("shared_and_self: contiguous rows and 32-bit gates");
+    Tensor o = alloc(DType::F32, h.rows(), h.cols());
+    const auto& k = kernels::routed();
+    Timed t(*this, Other);
+    call(launches_, k, k.shared_and_self(residual ? (const float*)residual->data : nullptr, shared ? (const float*)shared->data : nullptr,
+                                         logits ? (const float*)logits->data + gate_col : nullptr, logits ? (int)logits->ld : 0,
+                                         self ? (const float*)self->data : nullptr, h.data, (float*)o.data, (int)h.rows(), (int)h.cols(), code(h.dtype),
+                                         stream_), "shared_and_self");
+    return o;
+}
+
 void Ops::scale_by_route(Tensor& act, const Tensor& dense, int experts, int inner) {
     if (!act.contiguous() || act.cols() != (int64_t)experts * inner || dense.rows() != act.rows()) throw KernelError("scale_by_route: shapes");
     const auto& k = kernels::routed();
@@ -819,14 +899,15 @@ void Ops::scale_by_route(Tensor& act, const Tensor& dense, int experts, int inne
          "scale_by_route");
 }
 
-Tensor Ops::expert_gate_up(const Tensor& h, const Routing& r, const Tensor& w_gate_up, int top, int inner) {
+Tensor Ops::expert_gate_up(const Tensor& h, const Routing& r, const Tensor& w_gate_up, int top, int inner, int unit, float limit, float slope) {
     if (!h.contiguous() || h.dtype != w_gate_up.dtype || !w_gate_up.contiguous() || w_gate_up.cols() != h.cols())
         throw KernelError("expert_gate_up: rows and stacked gate/up weights of one dtype and width");
     Tensor act = alloc(h.dtype, h.rows() * top, inner);
     const auto& k = kernels::routed();
     Timed t(*this, Product);
     call(launches_, k, k.gate_up(h.data, (const int*)r.ids.data, w_gate_up.data, act.data, (int)h.rows(), top,
-                                 (int)(w_gate_up.rows() / (2 * (int64_t)inner)), (int)h.cols(), inner, code(h.dtype), stream_), "gate_up");
+                                 (int)(w_gate_up.rows() / (2 * (int64_t)inner)), (int)h.cols(), inner, unit, limit, slope, code(h.dtype),
+                                 stream_), "gate_up");
     return act;
 }
 
@@ -846,7 +927,7 @@ Tensor Ops::expert_down_combine(const Tensor& act, const Routing& r, const Tenso
 }
 
 Tensor Ops::experts_grouped(const Tensor& h, const Routing& r, const Tensor& w_gate_up, const Tensor& w_down, const Tensor& residual,
-                            int top, int inner) {
+                            int top, int inner, int unit, float limit, float slope) {
     const int64_t rows = h.rows(), width = h.cols(), n_pairs = rows * top;
     const int experts = (int)(w_gate_up.rows() / (2 * (int64_t)inner));
     const auto& k = kernels::routed();
@@ -860,12 +941,13 @@ Tensor Ops::experts_grouped(const Tensor& h, const Routing& r, const Tensor& w_g
     std::vector<int> off((size_t)experts + 1);
     cuda_check(cudaMemcpyAsync(off.data(), offsets, off.size() * sizeof(int), cudaMemcpyDeviceToHost, stream_), "cudaMemcpyAsync");
     cuda_check(cudaStreamSynchronize(stream_), "cudaStreamSynchronize");
-    Tensor gathered = gather_rows(row_at, n_pairs, h);
+    // (fewer places than pairs where some choices are no expert of this table: only the places that exist are gathered)
+    Tensor gathered = off.back() > 0 ? gather_rows(row_at, off.back(), h) : Tensor();
     Tensor part = alloc(DType::F32, n_pairs, width);
     for (int e = 0; e < experts; ++e) {
         const int64_t lo = off[(size_t)e], n = off[(size_t)e + 1] - lo;
         if (n <= 0) continue;
-        Tensor act = linear_swiglu(Rows(gathered.row_slice(lo, n)), w_gate_up.row_slice((int64_t)e * 2 * inner, 2 * (int64_t)inner));
+        Tensor act = linear_swiglu(Rows(gathered.row_slice(lo, n)), w_gate_up.row_slice((int64_t)e * 2 * inner, 2 * (int64_t)inner), unit, limit, slope);
         Tensor wd = w_down;                          // this expert's columns, the matrix's row stride
         wd.data = (char*)w_down.data + (size_t)e * inner * dtype_size(w_down.dtype);
         wd.shape[1] = inner;
@@ -1076,7 +1158,7 @@ Tensor Ops::qkv_rope_write(const Rows& x, const Tensor& weight, const Tensor* bi
     return qkv;
 }
 
-Tensor Ops::linear_swiglu(const Rows& x, const Tensor& weight_pairs, int act) {
+Tensor Ops::linear_swiglu(const Rows& x, const Tensor& weight_pairs, int act, float limit, float slope) {
     const Tensor& xt = x.t;
     check_product(xt, weight_pairs);
     const int64_t inner = weight_pairs.rows() / 2;
@@ -1086,9 +1168,27 @@ Tensor Ops::linear_swiglu(const Rows& x, const Tensor& weight_pairs, int act) {
         GemmFusion f;
         memset(&f, 0, sizeof f);
         fusion_in(x, f);
-        return linear_tc(xt, weight_pairs, nullptr, nullptr, out, -1, -1, -1, act, x.deferred ? &f : nullptr);
+        f.act_limit = limit;
+        f.act_slope = slope;
+        return linear_tc(xt, weight_pairs, nullptr, nullptr, out, -1, -1, -1, act, x.deferred || act == 3 ? &f : nullptr);
     }
-    return swiglu(linear(x, weight_pairs), act);
+    return swiglu(linear(x, weight_pairs), act, limit, slope);
+}
+
+Tensor Ops::linear_relu_squared(const Rows& x, const Tensor& weight) {
+    const Tensor& xt = x.t;
+    check_product(xt, weight);
+    Tensor probe = Tensor::make((void*)16, xt.dtype, {xt.rows(), weight.rows()});
+    if (xt.dtype == DType::BF16 && tensor_core_ok(xt, weight, probe, nullptr)) {
+        Tensor out = alloc(xt.dtype, xt.rows(), weight.rows());
+        GemmFusion f;
+        memset(&f, 0, sizeof f);
+        fusion_in(x, f);
+        return linear_tc(xt, weight, nullptr, nullptr, out, -1, -1, -1, 4, x.deferred ? &f : nullptr);
+    }
+    Tensor z = linear(x, weight);
+    relu_squared(z);
+    return z;
 }
 
 // ------------------------------------------------------------------ attention

@@ -256,6 +256,15 @@ private:
     std::string name_, bias_name_;
 };
 
+// ------------------------------------------------------------------ no norm
+// The rows themselves, in the activation dtype: what a sublayer reads whose block norms its result only.
+class IdentityNorm : public Norm {
+public:
+    IdentityNorm(const PartSpec&, const BuildEnv& e) : Norm(e) {}
+    Tensor forward(Ops& ops, const Tensor& x) override { return ops.cast_rows(x, env.dtype); }
+    bool identity() const override { return true; }
+};
+
 // ------------------------------------------------------------------ rotary encoding, NeoX pairing
 // The pair (i, i + rotary_dim/2) of every query and key head is rotated by the angle pos / theta^(2i / rotary_dim).
 // The angle is formed as the reference forms it (cuda_math_kernels.cu:337-339, cpu_ops.cpp:26-30): the denominator
@@ -721,6 +730,7 @@ private:
 namespace {
 PartRegistrar r1("norm", "rmsnorm", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new RMSNorm(s, e); });
 PartRegistrar r1b("norm", "layernorm", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new LayerNorm(s, e); });
+PartRegistrar r1c("norm", "identity", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new IdentityNorm(s, e); });
 PartRegistrar r2b("position", "rotary_pairs", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new RotaryPairs(s, e); });
 PartRegistrar r2("position", "rotary_neox", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new RotaryNeox(s, e); });
 PartRegistrar r3("position", "none", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new NoPosition(s, e); });

@@ -10,7 +10,11 @@
 //                              values as the cache keeps them; scores (q . k) * "scale", times 1 + coef * ln(floor((i + 1) /
 //                              every) + 1) with "q_temp": {coef, every}; "sink": exp(sink_h) joins head h's denominator
 //                              (tensor "sink" [heads]); then Wo.  The cache keeps the window's keys and values per token and,
-//                              with pooled blocks, a 32-bit row of sums per block.
+//                              with pooled blocks, a 32-bit row of sums per block.  More options: "qkv_bias" (tensors "q.b", "k.b",
+//                              "v.b"); "qk_norm": "whole" norms all query heads of a row at once (weights [heads * dim]),
+//                              likewise the keys; "softcap" c: score <- c tanh(score / c); "head_gate": head h's result is
+//                              multiplied by sigmoid(Wg h)_h (tensor "g" [heads, width]); "shared_kv": no keys and values of its
+//                              own (nor their norm), it reads the cache entry of an earlier layer.
 //   mixer "general_delta"      r, k, v = W h (heads x dim); decay w = exp(-rate * sigmoid(Ww2 tanh(Ww1 h) + w0)) and removal
 //                              a = sigmoid(Wa h + a.b) per head and key channel; with the unit key u = k / sqrt(sum k^2 + 1e-6):
 //                              S <- diag(w) S - (a u)(u^T S) + k v^T (both terms read the old S), o = S^T r; every head's o
@@ -68,13 +72,23 @@ public:
         scale_ = (float)s.params.get_double("scale", 1.0 / sqrt((double)dim_));
         eps_ = (float)s.params.get_double("eps", 1e-5);
         has_sink_ = s.params.get_bool("sink", false);
-        qk_norm_ = s.params.get_bool("qk_norm", false);
+        const Json* qn = s.params.find("qk_norm");
+        if (qn && !qn->is_bool() && !(qn->is_string() && (qn->as_string() == "heads" || qn->as_string() == "whole")))
+            throw ConfigError("pooled_attention: 'qk_norm' is true, false, \"heads\" or \"whole\"");
+        norm_whole_ = qn && qn->is_string() && qn->as_string() == "whole";
+        qk_norm_ = norm_whole_ || (qn && (qn->is_string() || qn->as_bool()));
+        softcap_ = (float)s.params.get_double("softcap", 0.0);
+        bias_ = s.params.get_bool("qkv_bias", false);
+        head_gate_ = s.params.get_bool("head_gate", false);
+        reads_ = s.params.get_bool("shared_kv", false);
         const std::string values = s.params.get_string("values", "own");
         if (values != "own" && values != "keys") throw ConfigError("pooled_attention: 'values' is \"own\" or \"keys\"");
         shared_ = values == "keys";
         if (kv_heads_ <= 0 || heads_ % kv_heads_) throw ConfigError(format("pooled_attention: %d heads cannot share %d key/value heads", heads_, kv_heads_));
         if (dim_ > 256 || vdim_ <= 0 || vdim_ > 256) throw ConfigError("pooled_attention: head sizes of 1 to 256");
         if (shared_ && vdim_ != dim_) throw ConfigError(format("pooled_attention: values that are the keys have the keys' size (dim %d, vdim %d)", dim_, vdim_));
+        if (softcap_ < 0.f) throw ConfigError("pooled_attention: 'softcap' must not be negative");
+        if (reads_ && (shared_ || pool_ > 0)) throw ConfigError("pooled_attention: a layer that reads another's keys and values has values of its own kind and no pooled blocks");
         if (window_ < 0 || pool_ < 0) throw ConfigError("pooled_attention: 'window' and 'pool' must not be negative");
         if (pool_ > 0 && window_ == 0) throw ConfigError("pooled_attention: pooled blocks lie before a window; without a window every token is seen");
         const Json* qt = s.params.find("q_temp");
@@ -84,14 +98,24 @@ public:
             if (temp_every_ <= 0) throw ConfigError("pooled_attention: 'q_temp' needs a positive 'every'");
         }
         position_ = adopt("", build<Position>("position", s.part("position"), e));
-        const int64_t w = e.width, qd = (int64_t)heads_ * dim_, kd = (int64_t)kv_heads_ * dim_, vd = shared_ ? 0 : (int64_t)kv_heads_ * vdim_;
-        declare_stacked("w_in", qd + kd + vd, w);
+        const int64_t w = e.width, qd = (int64_t)heads_ * dim_, kd = reads_ ? 0 : (int64_t)kv_heads_ * dim_;
+        const int64_t vd = shared_ || reads_ ? 0 : (int64_t)kv_heads_ * vdim_, gd = head_gate_ ? heads_ : 0;
+        // one product for queries, keys, values and gates; its columns are padded to whole 16-byte pieces, since the rows' queries
+        // and values are read as such
+        declare_stacked("w_in", (qd + kd + vd + gd + 7) / 8 * 8, w);
         declare("q", {qd, w}).stack("w_in", 0);
-        declare("k", {kd, w}).stack("w_in", qd);
-        if (!shared_) declare("v", {vd, w}).stack("w_in", qd + kd);
+        if (kd) declare("k", {kd, w}).stack("w_in", qd);
+        if (vd) declare("v", {vd, w}).stack("w_in", qd + kd);
+        if (gd) declare("g", {gd, w}).stack("w_in", qd + kd + vd);
+        if (bias_) {                                             // the gates have none: their rows stay zero
+            declare_stacked("b_in", (qd + kd + vd + gd + 7) / 8 * 8, 1);
+            declare("q.b", {qd}).stack("b_in", 0);
+            if (kd) declare("k.b", {kd}).stack("b_in", qd);
+            if (vd) declare("v.b", {vd}).stack("b_in", qd + kd);
+        }
         if (qk_norm_) {
-            declare("q.norm", {(int64_t)dim_}, false, true);
-            declare("k.norm", {(int64_t)dim_}, false, true);
+            declare("q.norm", {norm_whole_ ? qd : (int64_t)dim_}, false, true);
+            if (kd) declare("k.norm", {norm_whole_ ? kd : (int64_t)dim_}, false, true);
         }
         if (has_sink_) declare("sink", {(int64_t)heads_});
         declare("o", {w, (int64_t)heads_ * vdim_});
@@ -110,10 +134,12 @@ public:
         Mixer::finalize(ops);
         const float* denominators = nullptr;
         int d = 0;
-        if (position_->halves(&freq_, &rot_mult_, &rot_)) {
+        neighbours_ = position_->pairs(&freq_, &rot_mult_, &rot_);
+        if (neighbours_ || position_->halves(&freq_, &rot_mult_, &rot_)) {
             if (rot_ > dim_ || rot_ % 2) throw ConfigError(format("%s: %d rotated numbers in heads of %d", prefix.c_str(), rot_, dim_));
-        } else if (position_->rotary(&denominators, &d) || position_->pairs(&freq_, &rot_mult_, &d)) {
-            throw ConfigError(prefix + ": pooled_attention takes a position part that turns the pairs (i, i + dims / 2), or none");
+            if (norm_whole_ && !neighbours_) throw ConfigError(prefix + ": a norm over all heads at once goes with neighbouring pairs, or no rotation");
+        } else if (position_->rotary(&denominators, &d)) {
+            throw ConfigError(prefix + ": pooled_attention takes a position part with a table of frequencies, or none");
         }
     }
 
@@ -125,7 +151,12 @@ public:
             tokens = &view.parts[0];
             blocks = &view.parts[1];
         }
-        Tensor in = ops.linear(h, tensor("w_in"));
+        Tensor bias_flat;
+        if (bias_) {
+            const Tensor& b = tensor("b_in");
+            bias_flat = Tensor::make(b.data, b.dtype, {b.numel()});
+        }
+        Tensor in = ops.linear(h, tensor("w_in"), bias_ ? &bias_flat : nullptr);
         Ops::PooledSpec sp;
         sp.heads = heads_;
         sp.kv_heads = kv_heads_;
@@ -138,14 +169,19 @@ public:
         sp.temp_every = temp_every_;
         sp.sink = has_sink_ ? &tensor("sink") : nullptr;
         sp.q_norm = qk_norm_ ? &tensor("q.norm") : nullptr;
-        sp.k_norm = qk_norm_ ? &tensor("k.norm") : nullptr;
+        sp.k_norm = qk_norm_ && !reads_ ? &tensor("k.norm") : nullptr;
+        sp.norm_whole = norm_whole_;
         sp.eps = eps_;
         sp.freq = freq_;
         sp.rot_mult = rot_mult_;
         sp.rot = rot_;
+        sp.neighbours = neighbours_;
+        sp.softcap = softcap_;
+        const int64_t qd = (int64_t)heads_ * dim_, kd = reads_ ? 0 : (int64_t)kv_heads_ * dim_, vd = shared_ || reads_ ? 0 : (int64_t)kv_heads_ * vdim_;
         sp.q_off = 0;
-        sp.k_off = (int64_t)heads_ * dim_;
-        sp.v_off = shared_ ? -1 : sp.k_off + (int64_t)kv_heads_ * dim_;
+        sp.k_off = reads_ ? -1 : qd;
+        sp.v_off = shared_ ? -1 : qd + kd;
+        sp.gate_off = head_gate_ ? qd + kd + vd : -1;
         ops.pooled_store(in, sp, *tokens, blocks, ctx);
         Tensor mixed = ops.pooled_attention(in, sp, *tokens, blocks, ctx);
         return project_out(ops, mixed, tensor("o"), residual, out_scale);
@@ -153,8 +189,8 @@ public:
 
 private:
     int heads_, kv_heads_, dim_, vdim_, window_, pool_, temp_every_ = 0, rot_ = 0;
-    float scale_, eps_, temp_coef_ = 0.f, rot_mult_ = 1.0f;
-    bool has_sink_, qk_norm_, shared_;
+    float scale_, eps_, temp_coef_ = 0.f, rot_mult_ = 1.0f, softcap_ = 0.f;
+    bool has_sink_, qk_norm_, shared_, norm_whole_ = false, bias_ = false, head_gate_ = false, reads_ = false, neighbours_ = false;
     Position* position_;
     const float* freq_ = nullptr;
 };

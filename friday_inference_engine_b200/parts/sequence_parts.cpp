@@ -2,13 +2,15 @@
 // from token to token, a mixer that runs others side by side, routed experts, and a per-layer token input.
 //
 //   mixer "gated_linear_attention"   S_t = diag(a_t) S_(t-1) + k_t v_t^T,  o_t = S_t^T q_t,  a_t = sigmoid(z_t)^(1/tau)
+//   mixer "decayed_linear_attention" S_t = decay_h S_(t-1) + k_t v_t^T,  o_t = S_t^T q_t, q, k and v through silu
 //   mixer "shift_decay_mix"          each projection reads its own blend of the row and the row before it;
 //                                    o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t,  S_t = diag(w_t) S_(t-1) + k_t v_t^T,
 //                                    w_t = exp(-exp(z_t))
 //   mixer "parallel"                 sum of scale_i * mixer_i(h) over members that read the same input, each with a cache
 //                                    entry part of its own
 //   feed_forward "routed_experts"    top-k of a biased router, weights by softmax over the chosen logits, gated experts; or
-//                                    sigmoid scores with a choice bias and groups of experts, and an expert for every row
+//                                    sigmoid scores with a choice bias and groups of experts, or softmax scores with a choice bias
+//                                    and experts that return their input; and an expert for every row
 //   token_input "gated_token_table"  x += norm(proj(gelu_tanh(gate x) * table[token]))
 //
 // The states, the decays and everything that enters the recurrences besides the projections are fp32 (csrc/recurrence.cu);
@@ -104,6 +106,67 @@ private:
     int heads_, dk_, dv_;
     int64_t rank_;
     float tau_, eps_;
+};
+
+// ------------------------------------------------------------------ linear attention with a constant decay per head
+// q = silu(Wq h), k = silu(Wk h) (heads x dim), v = silu(Wv h) (heads x vdim); per head S = decay_h S + k v^T, o = S^T q with no
+// other scale ("decay": a number per head); the heads' results side by side are RMS-normed as one row with the weight "norm",
+// multiplied by sigmoid(Wg h) and projected by Wo.  State per sequence: the heads' matrices, fp32.
+class DecayedLinearAttention : public Mixer {
+public:
+    DecayedLinearAttention(const PartSpec& s, const BuildEnv& e) : Mixer(e) {
+        heads_ = positive(s, "heads", "decayed_linear_attention");
+        dk_ = positive(s, "dim", "decayed_linear_attention");
+        dv_ = (int)s.params.get_int("vdim", dk_);
+        eps_ = (float)s.params.get_double("eps", 1e-5);
+        const Json* d = s.params.find("decay");
+        if (!d || !d->is_array() || (int)d->size() != heads_) throw ConfigError("decayed_linear_attention needs 'decay', a number per head");
+        for (size_t i = 0; i < d->size(); ++i) table_.push_back((float)(*d)[i].as_double());
+        if (dv_ <= 0 || dk_ > 256) throw ConfigError("decayed_linear_attention: key sizes of 1 to 256 and a positive value size");
+        const int64_t w = e.width, hk = (int64_t)heads_ * dk_, hv = (int64_t)heads_ * dv_;
+        declare_stacked("w_in", (2 * hk + 2 * hv + 7) / 8 * 8, w);
+        declare("q", {hk, w}).stack("w_in", 0);
+        declare("k", {hk, w}).stack("w_in", hk);
+        declare("v", {hv, w}).stack("w_in", 2 * hk);
+        declare("g", {hv, w}).stack("w_in", 2 * hk + hv);
+        declare("norm", {hv}, false, true);
+        declare("o", {w, hv});
+    }
+    CacheRequest cache_request() const override { return CacheRequest::state({(int64_t)heads_ * dk_ * dv_}, DType::F32); }
+    void finalize(Ops& ops) override {
+        Mixer::finalize(ops);
+        auto mem = std::make_shared<DeviceBuffer>(table_.size() * sizeof(float));
+        cuda_check(cudaMemcpyAsync(mem->get(), table_.data(), table_.size() * sizeof(float), cudaMemcpyHostToDevice, ops.stream()),
+                   "cudaMemcpyAsync");
+        cuda_check(cudaStreamSynchronize(ops.stream()), "cudaStreamSynchronize");
+        decay_ = (const float*)mem->get();
+        hold(mem);
+    }
+
+    PartOut forward(Ops& ops, const Rows& h, const Tensor& residual, const StepContext& ctx, const CacheView& view, Norm*) override {
+        const int64_t hk = (int64_t)heads_ * dk_, hv = (int64_t)heads_ * dv_;
+        Tensor in = ops.linear(h, tensor("w_in"));
+        Ops::DecaySpec sp;
+        sp.heads = heads_;
+        sp.dk = dk_;
+        sp.dv = dv_;
+        sp.decay = decay_;
+        sp.q_off = 0;
+        sp.k_off = hk;
+        sp.v_off = 2 * hk;
+        Tensor o = ops.decay_scan(in, sp, view, ctx);
+        Tensor y = ops.row_norm_gate(o, columns(in, 2 * hk + hv, hv), tensor("norm"), eps_, in.dtype);
+        if (residual.defined()) return PartOut(ops.linear_residual(Rows(y), tensor("o"), nullptr, residual, out_scale));
+        Tensor out = ops.linear(Rows(y), tensor("o"), nullptr, nullptr, (int)DType::F32);        // the block sums itself
+        if (out_scale != 1.0f) ops.scale_rows(out, out_scale);
+        return PartOut(out);
+    }
+
+private:
+    int heads_, dk_, dv_;
+    float eps_;
+    std::vector<float> table_;
+    const float* decay_ = nullptr;
 };
 
 // ------------------------------------------------------------------ token-shift mixing with a data-dependent decay
@@ -266,30 +329,54 @@ public:
         top_ = positive(s, "top", "routed_experts");
         inner_ = positive(s, "inner", "routed_experts");
         softmax_all_ = s.params.get_bool("softmax_all", false);
-        if (top_ > experts_) throw ConfigError(format("routed_experts: top %d of %d experts", top_, experts_));
+        if (top_ > experts_ + (int)s.params.get_int("identity", 0)) throw ConfigError(format("routed_experts: top %d of %d experts", top_, experts_));
         if (top_ > 32 || experts_ > 256) throw ConfigError("routed_experts: at most 256 experts and 32 choices");
         // "score": "sigmoid" makes the scores sigmoid(logit): the choice runs on score + the tensor "choice_bias" (if named)
         // among the experts of the "groups_keep" best of "groups" equally sized runs of adjacent experts (a group counts as the sum of its
         // two largest), the weights are score * "weight_scale", not renormalised.  "router_bias": false leaves the logits'
         // bias out.  "shared_inner" > 0 adds an expert of that inner size ("shared.") that every row uses.
+        // "score": "softmax_biased" makes the scores the softmax over everything the router knows: the experts and "identity" more
+        // outputs whose experts return their input; the choice runs on score + the tensor "choice_bias", the weights are the
+        // chosen scores divided by their sum.  "activation": "silu" (gate times up), or "clipped" with "limit" L and "slope" a:
+        // g sigmoid(a g) (u + 1), g = min(gate, L), u = clamp(up, -L, L) ("shared_limit": the L of the expert that every row
+        // uses).  "shared_gate" names a row [1, width] whose sigmoid multiplies that expert's result.
         const std::string score = s.params.get_string("score", "softmax");
-        if (score != "softmax" && score != "sigmoid") throw ConfigError("routed_experts: 'score' is \"softmax\" or \"sigmoid\"");
+        if (score != "softmax" && score != "sigmoid" && score != "softmax_biased")
+            throw ConfigError("routed_experts: 'score' is \"softmax\", \"sigmoid\" or \"softmax_biased\"");
         sigmoid_ = score == "sigmoid";
+        biased_ = score == "softmax_biased";
+        identity_ = (int)s.params.get_int("identity", 0);
+        if (identity_ < 0 || (identity_ > 0 && !biased_) || experts_ + identity_ > 256)
+            throw ConfigError("routed_experts: experts that return their input belong to biased softmax scores, 256 experts in all");
+        const std::string act = s.params.get_string("activation", "silu");
+        if (act != "silu" && act != "clipped") throw ConfigError("routed_experts: 'activation' is \"silu\" or \"clipped\"");
+        act_ = act == "clipped" ? 3 : 1;
+        limit_ = (float)s.params.get_double("limit", 0.0);
+        shared_limit_ = (float)s.params.get_double("shared_limit", limit_);
+        slope_ = (float)s.params.get_double("slope", 1.0);
+        shared_gate_ = s.params.get_string("shared_gate", "");
         router_bias_ = s.params.get_bool("router_bias", true);
         choice_bias_ = s.params.get_string("choice_bias", "");
         groups_ = (int)s.params.get_int("groups", 1);
         keep_ = (int)s.params.get_int("groups_keep", groups_);
         weight_scale_ = (float)s.params.get_double("weight_scale", 1.0);
         shared_inner_ = s.params.get_int("shared_inner", 0);
-        if (groups_ < 1 || experts_ % groups_ || keep_ < 1 || keep_ > groups_ || keep_ * (experts_ / groups_) < top_)
+        if (groups_ < 1 || experts_ % groups_ || keep_ < 1 || keep_ > groups_ || keep_ * (experts_ / groups_) + identity_ < top_)
             throw ConfigError(format("routed_experts: %d experts in %d groups of which %d are kept cannot give %d choices", experts_,
                                      groups_, keep_, top_));
-        if (!sigmoid_ && (groups_ > 1 || !choice_bias_.empty() || weight_scale_ != 1.0f))
+        if (!sigmoid_ && (groups_ > 1 || (!biased_ && !choice_bias_.empty()) || weight_scale_ != 1.0f))
             throw ConfigError("routed_experts: groups, a choice bias and a weight multiplier belong to sigmoid scores");
-        const int64_t w = e.width;
-        declare("router", {(int64_t)experts_, w});
-        if (router_bias_) declare("router.b", {(int64_t)experts_});
-        if (!choice_bias_.empty()) declare(choice_bias_, {(int64_t)experts_});
+        if (!shared_gate_.empty() && (shared_inner_ <= 0 || router_bias_)) throw ConfigError("routed_experts: 'shared_gate' belongs to an expert that every row uses and a router without bias");
+        const int64_t w = e.width, outputs = (int64_t)experts_ + identity_;
+        if (shared_gate_.empty()) {
+            declare("router", {outputs, w});
+        } else {                                                 // the gate is one more row of the router's product
+            declare_stacked("w_router", outputs + 1, w);
+            declare("router", {outputs, w}).stack("w_router", 0);
+            declare(shared_gate_, {1, w}).stack("w_router", outputs);
+        }
+        if (router_bias_) declare("router.b", {outputs});
+        if (!choice_bias_.empty()) declare(choice_bias_, {outputs});
         if (shared_inner_ > 0) {
             declare_stacked("w_shared", 2 * shared_inner_, w);
             declare("shared.gate", {shared_inner_, w}).stack("w_shared", 0, 2);
@@ -307,12 +394,14 @@ public:
     }
     PartOut forward(Ops& ops, const Rows& h, const Tensor& residual_in, const StepContext& ctx, Norm*) override {
         Tensor x = ops.materialize(h);
-        Tensor logits = ops.linear(Rows(x), tensor("router"), router_bias_ ? &tensor("router.b") : nullptr, nullptr, (int)DType::F32);
+        Tensor logits = ops.linear(Rows(x), tensor(shared_gate_.empty() ? "router" : "w_router"), router_bias_ ? &tensor("router.b") : nullptr, nullptr, (int)DType::F32);
         // what the chosen experts' results are added to: the stream; with an expert that every row uses, its result on top
         // of the stream; without a stream (a block that sums itself), that result alone or zeros, 32-bit
         Tensor residual = residual_in;
-        if (shared_inner_ > 0) {
-            Tensor act = ops.linear_swiglu(Rows(x), tensor("w_shared"));
+        if (biased_) {
+            // (below: gated by the row's own gate and with the share of the experts that return their input, once the choice is known)
+        } else if (shared_inner_ > 0) {
+            Tensor act = ops.linear_swiglu(Rows(x), tensor("w_shared"), act_, shared_limit_, slope_);
             if (residual.defined()) residual = ops.linear_residual(Rows(act), tensor("shared.down"), nullptr, residual);
             else residual = ops.linear(Rows(act), tensor("shared.down"), nullptr, nullptr, (int)DType::F32);
         } else if (!residual.defined()) {
@@ -337,21 +426,36 @@ public:
         const bool dense = tensor_cores && !grouped && (forced == "dense" || (forced.empty() && experts_ <= 16 * top_));
         Ops::Routing r = sigmoid_ ? ops.route_scored(logits, top_, choice_bias_.empty() ? nullptr : &tensor(choice_bias_), groups_, keep_,
                                                      weight_scale_, dense)
+                        : biased_ ? ops.route_biased(logits, experts_, identity_, top_, choice_bias_.empty() ? nullptr : &tensor(choice_bias_), dense)
                                   : ops.route(logits, top_, softmax_all_, dense);
-        if (grouped) return PartOut(ops.experts_grouped(x, r, tensor("w_gate_up"), tensor("w_down"), residual, top_, inner_));
+        if (biased_) {
+            Tensor shared;
+            if (shared_inner_ > 0) {
+                Tensor act = ops.linear_swiglu(Rows(x), tensor("w_shared"), act_, shared_limit_, slope_);
+                shared = ops.linear(Rows(act), tensor("shared.down"), nullptr, nullptr, (int)DType::F32);
+            }
+            residual = ops.shared_and_self(residual_in.defined() ? &residual_in : nullptr, shared.defined() ? &shared : nullptr,
+                                           shared_gate_.empty() ? nullptr : &logits, (int64_t)experts_ + identity_,
+                                           r.self.defined() ? &r.self : nullptr, x);
+        }
+        if (grouped)
+            return PartOut(ops.experts_grouped(x, r, tensor("w_gate_up"), tensor("w_down"), residual, top_, inner_, act_, limit_, slope_));
         if (dense) {
-            Tensor act = ops.linear_swiglu(Rows(x), tensor("w_gate_up"));
+            Tensor act = ops.linear_swiglu(Rows(x), tensor("w_gate_up"), act_, limit_, slope_);
             ops.scale_by_route(act, r.dense, experts_, inner_);
             return PartOut(ops.linear_residual(Rows(act), tensor("w_down"), nullptr, residual));
         }
-        Tensor act = ops.expert_gate_up(x, r, tensor("w_gate_up"), top_, inner_);
+        Tensor act = ops.expert_gate_up(x, r, tensor("w_gate_up"), top_, inner_, act_, limit_, slope_);
         return PartOut(ops.expert_down_combine(act, r, tensor("w_down"), residual, top_, inner_));
     }
 
 private:
     int experts_, top_, inner_;
     bool softmax_all_;
-    bool sigmoid_ = false, router_bias_ = true;
+    bool sigmoid_ = false, router_bias_ = true, biased_ = false;
+    int identity_ = 0, act_ = 1;
+    float limit_ = 0.f, shared_limit_ = 0.f, slope_ = 1.f;
+    std::string shared_gate_;
     std::string choice_bias_;
     int groups_ = 1, keep_ = 1;
     float weight_scale_ = 1.0f;
@@ -394,6 +498,7 @@ private:
 
 namespace {
 PartRegistrar s1("mixer", "gated_linear_attention", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new GatedLinearAttention(s, e); });
+PartRegistrar s1b("mixer", "decayed_linear_attention", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new DecayedLinearAttention(s, e); });
 PartRegistrar s2("mixer", "shift_decay_mix", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new ShiftDecayMix(s, e); });
 PartRegistrar s3("mixer", "parallel", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new ParallelMixer(s, e); });
 PartRegistrar s4("feed_forward", "routed_experts", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new RoutedExperts(s, e); });
