@@ -697,6 +697,64 @@ def vulanex_numbers(cfg, batch, context, prompt_len):
     return {"step_bytes": weight_bytes + state_bytes + kv_bytes, "flops_per_token": flops}
 
 
+def zudovik_config(width, layers=7, vocab=32768, experts=8, top=2):
+    """A Zudovik configuration whose layers have sizes like a real model's of this width: in turn attention with keys and values
+    of its own, linear attention with heads of 128 x 128, and attention with keys and values of its own that the layer after it
+    reads too; heads of 128 on a quarter as many key/value heads, half of a head rotated; a dense feed-forward of four times
+    the width in the even layers and, in the odd ones, `experts` experts of inner size width and one that returns its input, `top`
+    of them chosen, with an expert of that size that every token uses."""
+    heads, kv = max(1, width // 128), max(1, width // 512)
+    att = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0, "rot": {"base": 10000.0, "dims": 64}}
+    lin = {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(3.0 + 7.0 * h / heads) for h in range(heads)]}
+    dense = {"kind": "dense", "ff": 4 * width}
+    moe = {"kind": "moe", "expert": {"ff": width, "limit": 7.0}, "router": {"experts": experts, "identity": 1, "top": top},
+           "shared": {"ff": width, "limit": 7.0}}
+    ls = []
+    for i in range(layers):
+        if i % 3 == 1:
+            ls.append({"type": "lightning", "mixer": lin})
+        else:
+            ls.append({"type": "attention", "mixer": dict(att, kv_from=i - 1) if i % 3 == 0 and i > 0 else att})
+        ls[-1]["mlp"] = dense if i % 2 == 0 else moe
+    return {"architecture": "Zudovik", "vocab": vocab, "width": width, "embedding": {"scale": 12.0}, "norm": {"eps": 1e-6}, "layers": ls}
+
+
+def zudovik_numbers(cfg, batch, context, prompt_len):
+    """What a decode step of `batch` sequences must read (weights, the experts that the batch touches, cached keys and values once
+    per layer that reads them, the states) and what a prompt token costs (the attention's share for a prompt of prompt_len
+    tokens; the experts chosen only)."""
+    w, v = cfg["width"], cfg["vocab"]
+    weight_bytes = 2 * v * w
+    flops = 2 * v * w
+    state_bytes = kv_bytes = 0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        H, d, vd = m["heads"], m["dim"], m["vdim"]
+        if L["type"] == "lightning":
+            mat = 2 * H * (d + vd) * w + w * H * vd
+            state_bytes += batch * H * d * vd * 4 * 2
+            mix = 4 * H * d * vd
+        else:
+            G = m["kv_heads"]
+            mat = H * d * w + w * H * vd + H * w + (0 if m.get("kv_from") is not None else G * (d + vd) * w)
+            kv_bytes += batch * context * G * (d + vd) * 2
+            mix = 2 * H * (d + vd) * prompt_len // 2
+        ff = ff_read = 0
+        mlp = L.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            ff = ff_read = 2 * mlp["ff"] * w
+        elif mlp:
+            r, f = mlp["router"], 3 * mlp["expert"]["ff"] * w
+            total = r["experts"] + r["identity"]
+            chosen = r["top"] * r["experts"] / total
+            distinct = r["experts"] * (1.0 - (1.0 - r["top"] / total) ** batch)
+            base = total * w + (3 * mlp["shared"]["ff"] * w + w if mlp.get("shared") else 0)
+            ff, ff_read = base + chosen * f, base + distinct * f
+        weight_bytes += 2 * (mat + ff_read)
+        flops += 2 * (mat + ff) + mix
+    return {"step_bytes": weight_bytes + state_bytes + kv_bytes, "flops_per_token": flops}
+
+
 def tikunex_numbers(cfg, batch, context):
     """What a decode step of `batch` sequences must read and what a prompt token costs, per run of the layers."""
     w, v = cfg["width"], cfg["vocab"]
@@ -742,7 +800,7 @@ def tikunex_numbers(cfg, batch, context):
 
 
 def design_compare(Engine, args):
-    """Vulanex, Ditenex, Beletar and Tikunex beside the Qwen2.5 dense decoder at equal width and depth (random weights): one prompt and decode
+    """Zudovik, Vulanex, Ditenex, Beletar and Tikunex beside the Qwen2.5 dense decoder at equal width and depth (random weights): one prompt and decode
     steps, with the share of each kind of kernel in the prompt (event-bracketed).  One line of text per measurement.
     --designs picks among them."""
     pk = peaks()
@@ -750,6 +808,7 @@ def design_compare(Engine, args):
     for width in [int(v) for v in args.design_compare.split(",") if v]:
         layers = args.layers or 4
         designs = [
+            ("zudovik", zudovik_config(width, 2 * layers - 1)),
             ("vulanex", vulanex_config(width, 2 * layers - 1)),
             ("ditenex", ditenex_config(width, 2 * layers - 1)),
             ("beletar", beletar_config(width, layers)),
@@ -761,7 +820,10 @@ def design_compare(Engine, args):
             if name not in args.designs.split(","):
                 continue
             eng = Engine(config=cfg, seed=0, dtype="bfloat16", max_ctx=4096, max_batch=batch, max_tokens=batch * 4096 + 8192)
-            if name == "vulanex":
+            if name == "zudovik":
+                nums = zudovik_numbers(cfg, batch, context + 64, prompt_len)
+                flops_tok, step_bytes = nums["flops_per_token"], nums["step_bytes"]
+            elif name == "vulanex":
                 nums = vulanex_numbers(cfg, batch, context + 64, prompt_len)
                 flops_tok, step_bytes = nums["flops_per_token"], nums["step_bytes"]
             elif name == "ditenex":
@@ -834,9 +896,9 @@ def main():
     ap.add_argument("--prefill-chunk", type=int, default=0, dest="prefill_chunk",
                     help="most tokens of a sequence per pass in the sweeps (0: the engine's own)")
     ap.add_argument("--design-compare", default="", dest="design_compare",
-                    help="widths, e.g. 1024,2048,4096: a Vulanex, a Ditenex, a Beletar and a Tikunex model with layers of that size beside the Qwen2.5 "
+                    help="widths, e.g. 1024,2048,4096: a Zudovik, a Vulanex, a Ditenex, a Beletar and a Tikunex model with layers of that size beside the Qwen2.5 "
                          "decoder of equal width (prompt, decode steps, kernel shares): lines of text")
-    ap.add_argument("--designs", default="vulanex,ditenex,beletar,tikunex,qwen2", help="which designs --design-compare runs")
+    ap.add_argument("--designs", default="zudovik,vulanex,ditenex,beletar,tikunex,qwen2", help="which designs --design-compare runs")
     ap.add_argument("--timeline", action="store_true",
                     help="print the kernels of one decode step as they run inside the captured graph (torch profiler)")
     args = ap.parse_args()
