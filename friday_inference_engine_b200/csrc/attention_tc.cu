@@ -31,7 +31,13 @@
 // tokens) are launched first.  Every wait on an mbarrier is bounded (two seconds), then a code goes to `status` and
 // all roles leave their loops.
 //
-// Head sizes: multiples of 16 up to 128.  One-token steps keep the mma.sync kernel (attention_mma.cu), whose rows
+// Both kernels exist in a second form (EXTRA) for designs whose softmax has more to it: scores capped as c tanh(s / c), a
+// number per head whose exponential joins the denominator, a sigmoid gate per row and head on the result, and weights that stay
+// 32-bit in effect: P enters the second product as two bf16 numbers each, the head over the first half of its S's columns and
+// the remainder over the second half, with one product for each.  c tanh(s / c) = c - 2 c / (e^(2 s / c) + 1) costs one
+// exponential and one reciprocal per score; its absolute error is a few units in the last place of c, like the score's own.
+//
+// Head sizes: multiples of 16 up to 128, values of a size of their own.  One-token steps keep the mma.sync kernel (attention_mma.cu), whose rows
 // of a CTA share a token.
 #include <cuda.h>
 #include <math.h>
@@ -65,8 +71,13 @@ struct TcArgs {
     const int* seq_pos0;      // position of its first row
     const int* seq_live;      // may be null; < 0 at seq_start[s]: the sequence has ended
     int* status;
-    int table_width, nq, nkv, hd, window, pool_rows, n_seqs;
+    int table_width, nq, nkv, hd, vd, window, pool_rows, n_seqs;
     float scale_log2;         // softmax scale times log2(e)
+    // EXTRA only
+    FrVec sink;               // [nq]; p null: none
+    const bf16* gate;         // head h's gate of row r at gate[r * gate_ld + h]; null: none
+    int gate_ld;
+    float cap_log2, two_over_cap_log2;   // cap (0: none) and, times the scale, 2 / cap, both in units of log2
     unsigned long long* trace;   // for measurements (may be null): [cta][8] sums of time (ns) that row 0's thread spent
                                  // waiting for S, reading it, writing P, rescaling O, waiting for the last product;
                                  // then blocks, total time, start
@@ -125,6 +136,21 @@ __device__ __forceinline__ float exp2_fast(float x) {
     return y;
 }
 
+// a raw score as the softmax sees it, in units of log2: scaled, and capped if there is a cap
+__device__ __forceinline__ float scaled_capped(const TcArgs& p, float raw) {
+    if (p.cap_log2 <= 0.f) return raw * p.scale_log2;
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(exp2_fast(raw * p.two_over_cap_log2) + 1.0f));
+    return fmaf(-2.0f * p.cap_log2, r, p.cap_log2);
+}
+// what a row's sum must become for the sink and the gate: result = O * factor
+__device__ __forceinline__ float row_factor(const TcArgs& p, float l, float m, int row, int head) {
+    if (p.sink.p != nullptr) l += exp2f(fmaf(p.sink.at(head), LOG2E, -m));
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (p.gate != nullptr) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)row * p.gate_ld + head]));
+    return inv;
+}
+
 __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
@@ -139,6 +165,18 @@ __device__ __forceinline__ void tc_st16(uint32_t taddr, const uint32_t (&r)[16])
           "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
         : "memory");
 }
+// 32 scores (in units of log2) become weights 2^(s + neg_m), each as two bf16 numbers: the weight rounded, and what rounding left
+__device__ __forceinline__ void split_weights(const uint32_t* s, float neg_m, float (&sum4)[4], uint32_t (&head)[16], uint32_t (&rest)[16]) {
+#pragma unroll
+    for (int j = 0; j < 32; j += 2) {
+        const float e0 = exp2_fast(__uint_as_float(s[j]) + neg_m), e1 = exp2_fast(__uint_as_float(s[j + 1]) + neg_m);
+        sum4[j & 2] += e0;
+        sum4[(j & 2) + 1] += e1;
+        const uint32_t h = pack2(e0, e1);
+        head[j >> 1] = h;
+        rest[j >> 1] = pack2(e0 - __uint_as_float(h << 16), e1 - __uint_as_float(h & 0xffff0000u));
+    }
+}
 // D[tmem] (+)= A[tmem] * B[smem]: the A operand lies in tensor memory (lane = row, two bf16 per 32-bit column)
 __device__ __forceinline__ void tc_mma_ta(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
                                           uint32_t accumulate) {
@@ -149,6 +187,7 @@ __device__ __forceinline__ void tc_mma_ta(uint32_t d_tmem, uint32_t a_tmem, uint
         : "memory");
 }
 
+template <bool EXTRA>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const TcArgs p) {
@@ -187,7 +226,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int lo_min = p.window > 0 ? max(0, pos0 + t0 - p.window + 1) : 0;
     const int kb_begin = lo_min / KEYS, kb_end = pos_hi / KEYS;       // inclusive
     const int n_blocks = kb_end - kb_begin + 1;
-    const int slices = (p.hd + 63) / 64;
+    const int slices = (p.hd + 63) / 64, vslices = (p.vd + 63) / 64;
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
@@ -238,26 +277,26 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 return p.pool_rows;
             };
             // a stage is free again when the product that read it is done: K after the scores, V after the second product
-            auto load = [&](int i, const CUtensorMap* map, uint8_t* ring, uint32_t full, uint32_t empty) {
+            auto load = [&](int i, const CUtensorMap* map, int n_slices, uint8_t* ring, uint32_t full, uint32_t empty) {
                 const int b = i & 1, par = (i >> 1) & 1;
                 if (!mbar_wait(empty + 8 * b, par ^ 1, p.status, 1)) return false;
-                mbar_expect_tx(full + 8 * b, (uint32_t)slices * KSLICE);
+                mbar_expect_tx(full + 8 * b, (uint32_t)n_slices * KSLICE);
                 const int row = page_row(i);
-                for (int s = 0; s < slices; ++s)
+                for (int s = 0; s < n_slices; ++s)
                     tma_load_3d(smem_u32(ring) + (uint32_t)(b * KV_STAGE + s * KSLICE), map, s * 64, kvh, row, full + 8 * b);
                 return true;
             };
             // in the order in which the products want them: K of the block after, then V of this one
-            bool ok = load(0, &map_k, s_k, k_full, k_empty);
+            bool ok = load(0, &map_k, slices, s_k, k_full, k_empty);
             for (int i = 0; i < n_blocks && ok; ++i) {
-                if (i + 1 < n_blocks) ok = load(i + 1, &map_k, s_k, k_full, k_empty);
-                if (ok) ok = load(i, &map_v, s_v, v_full, v_empty);
+                if (i + 1 < n_blocks) ok = load(i + 1, &map_k, slices, s_k, k_full, k_empty);
+                if (ok) ok = load(i, &map_v, vslices, s_v, v_full, v_empty);
             }
         }
     } else if (warp == 1) {
         if (elect_one()) {
             const uint32_t idesc_qk = instr_desc(ROWS, KEYS);
-            const uint32_t idesc_pv = instr_desc(ROWS, p.hd) | (1u << 16);   // B is MN-major
+            const uint32_t idesc_pv = instr_desc(ROWS, p.vd) | (1u << 16);   // B is MN-major
             const int k_steps = p.hd / 16;                                   // of the first product
             bool ok = mbar_wait(q_full, 0, p.status, 2);
             unsigned long long m_spent[5] = {0, 0, 0, 0, 0}, m_mark = p.trace != nullptr ? global_ns() : 0;
@@ -303,6 +342,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 for (int ks = 0; ks < pv_steps; ++ks) {
                     const uint64_t db = smem_desc_mn(smem_u32(s_v) + b * KV_STAGE + ks * 16 * 128, KSLICE, 1024);
                     tc_mma_ta(tmem_o, tmem_s + b * KEYS + 8 * ks, db, idesc_pv, (i > 0 || ks > 0) ? 1u : 0u);
+                    if (EXTRA) tc_mma_ta(tmem_o, tmem_s + b * KEYS + KEYS / 2 + 8 * ks, db, idesc_pv, 1u);
                 }
                 tc_commit(pv_done + 8 * b);
                 tc_commit(v_empty + 8 * b);
@@ -363,6 +403,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             // The maximum of the raw scores in four strands (one strand of dependent comparisons would be paid in full:
             // a scheduler has few such warps to choose from); the positive scale is applied to the result.
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+            if (EXTRA) {                                   // scaled and capped here, in place
+#pragma unroll
+                for (int j = 0; j < KEYS; ++j) raw[j] = __float_as_uint(scaled_capped(p, __uint_as_float(raw[j])));
+            }
             if (need_mask) {
 #pragma unroll
                 for (int j = 0; j < KEYS; ++j) {
@@ -373,7 +417,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 #pragma unroll
                 for (int j = 0; j < KEYS; ++j) mx4[j & 3] = fmaxf(mx4[j & 3], __uint_as_float(raw[j]));
             }
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (EXTRA ? 1.f : p.scale_log2);
             lap(1);
             // The reference maximum moves only when the true one has grown by more than 8; O is rescaled then.
             // tcgen05.ld and .st are warp-wide, so a warp rescales if any of its rows must.
@@ -392,7 +436,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     tc_fence_after();
 #pragma unroll 1
                     for (int c = 0; c < 8; ++c) {
-                        if (c * 16 < p.hd) {
+                        if (c * 16 < p.vd) {
                             uint32_t o16[16];
                             tc_ld16(tmem_o + lane_addr + c * 16, o16);
                             tc_ld_wait();
@@ -409,16 +453,26 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             // -inf and stays so; a row that has seen no key takes its exponentials against 0.
             const float neg_m = m_run == -INFINITY ? 0.f : -m_run;
             float sum4[4] = {0.f, 0.f, 0.f, 0.f};            // four strands, for the same reason
-            uint32_t packed[KEYS / 2];
+            if (EXTRA) {
 #pragma unroll
-            for (int j = 0; j < KEYS; j += 2) {
-                const float e0 = exp2_fast(fmaf(__uint_as_float(raw[j]), p.scale_log2, neg_m));
-                const float e1 = exp2_fast(fmaf(__uint_as_float(raw[j + 1]), p.scale_log2, neg_m));
-                sum4[j & 2] += e0;
-                sum4[(j & 2) + 1] += e1;
-                packed[j >> 1] = pack2(e0, e1);
+                for (int h = 0; h < 2; ++h) {
+                    uint32_t head16[16], rest16[16];
+                    split_weights(&raw[32 * h], neg_m, sum4, head16, rest16);
+                    tc_st16(s_addr + 16 * h, head16);
+                    tc_st16(s_addr + KEYS / 2 + 16 * h, rest16);
+                }
+            } else {
+                uint32_t packed[KEYS / 2];
+#pragma unroll
+                for (int j = 0; j < KEYS; j += 2) {
+                    const float e0 = exp2_fast(fmaf(__uint_as_float(raw[j]), p.scale_log2, neg_m));
+                    const float e1 = exp2_fast(fmaf(__uint_as_float(raw[j + 1]), p.scale_log2, neg_m));
+                    sum4[j & 2] += e0;
+                    sum4[(j & 2) + 1] += e1;
+                    packed[j >> 1] = pack2(e0, e1);
+                }
+                tc_st32(s_addr, packed);
             }
-            tc_st32(s_addr, packed);
             tc_st_wait();
             l_run += (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]);
             if (kb == kb_end) {
@@ -426,7 +480,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 const int key = j0 + r;
                 if (r < KEYS && key > pos_hi) {
                     if (!(ok = mbar_wait(v_full + 8 * b, par, p.status, 7))) break;
-                    for (int s = 0; s < slices; ++s) {
+                    for (int s = 0; s < vslices; ++s) {
                         uint4* line = (uint4*)(s_v + b * KV_STAGE + s * KSLICE + r * 128);
 #pragma unroll
                         for (int q = 0; q < 8; ++q) line[q] = make_uint4(0u, 0u, 0u, 0u);
@@ -443,18 +497,18 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         tc_fence_after();
         lap(4);
         if (ok) {
-            const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-            bf16* dst = p.out + ((size_t)(q_start + t0 + t) * p.nq + (size_t)kvh * G + g) * p.hd;
+            const float inv = !valid ? 0.f : EXTRA ? row_factor(p, l_run, m_run, q_start + t0 + t, kvh * G + g) : l_run > 0.f ? 1.f / l_run : 0.f;
+            bf16* dst = p.out + ((size_t)(q_start + t0 + t) * p.nq + (size_t)kvh * G + g) * p.vd;
 #pragma unroll 1
             for (int c = 0; c < 4; ++c) {
-                if (c * 32 < p.hd) {                                   // uniform: the load is warp-wide
+                if (c * 32 < p.vd) {                                   // uniform: the load is warp-wide
                     uint32_t o32[32];
                     tc_ld32(tmem_o + lane_addr + c * 32, o32);
                     tc_ld_wait();
                     if (valid) {
 #pragma unroll
                         for (int q = 0; q < 4; ++q) {
-                            if (c * 32 + q * 8 < p.hd) {
+                            if (c * 32 + q * 8 < p.vd) {
                                 float x[8];
 #pragma unroll
                                 for (int j = 0; j < 8; ++j) x[j] = __uint_as_float(o32[q * 8 + j]) * inv;
@@ -501,6 +555,7 @@ constexpr int KSLICE2 = KEYS2 * 128;      // a block's keys (or values), 64 dims
 constexpr int KV_STAGE2 = 2 * KSLICE2;
 constexpr int SMEM_BYTES2 = 4 * SLICE + 4 * KV_STAGE2 + 1024 + 256;
 
+template <bool EXTRA>
 __global__ void __launch_bounds__(THREADS2, 1)
 attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const TcArgs p) {
@@ -544,7 +599,7 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int ub0 = kb0[0], ub1 = active[1] ? kb1[1] : kb1[0];
     const int n_blocks = ub1 - ub0 + 1;
     const int pos_hi_u = active[1] ? pos_hi[1] : pos_hi[0];
-    const int slices = (p.hd + 63) / 64;
+    const int slices = (p.hd + 63) / 64, vslices = (p.vd + 63) / 64;
     auto part = [&](int x, int i) { return active[x] && ub0 + i >= kb0[x] && ub0 + i <= kb1[x]; };
 
     if (threadIdx.x == 0) {
@@ -593,28 +648,28 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 }
                 return p.pool_rows;                    // beyond the pool: zeros
             };
-            auto load = [&](int i, const CUtensorMap* map, uint8_t* ring, uint32_t full, uint32_t empty) {
+            auto load = [&](int i, const CUtensorMap* map, int n_slices, uint8_t* ring, uint32_t full, uint32_t empty) {
                 const int b = i & 1, par = (i >> 1) & 1;
                 if (!mbar_wait(empty + 8 * b, par ^ 1, p.status, 1)) return false;
-                mbar_expect_tx(full + 8 * b, (uint32_t)(2 * slices * KSLICE));
+                mbar_expect_tx(full + 8 * b, (uint32_t)(2 * n_slices * KSLICE));
                 for (int pg = 0; pg < 2; ++pg) {
                     const int row = page_row(2 * (ub0 + i) + pg);
-                    for (int s = 0; s < slices; ++s)
+                    for (int s = 0; s < n_slices; ++s)
                         tma_load_3d(smem_u32(ring) + (uint32_t)(b * KV_STAGE2 + s * KSLICE2 + pg * KSLICE), map, s * 64, kvh, row,
                                     full + 8 * b);
                 }
                 return true;
             };
-            bool ok = load(0, &map_k, s_k, k_full, k_empty);
+            bool ok = load(0, &map_k, slices, s_k, k_full, k_empty);
             for (int i = 0; i < n_blocks && ok; ++i) {
-                if (i + 1 < n_blocks) ok = load(i + 1, &map_k, s_k, k_full, k_empty);
-                if (ok) ok = load(i, &map_v, s_v, v_full, v_empty);
+                if (i + 1 < n_blocks) ok = load(i + 1, &map_k, slices, s_k, k_full, k_empty);
+                if (ok) ok = load(i, &map_v, vslices, s_v, v_full, v_empty);
             }
         }
     } else if (warp == 1) {
         if (elect_one()) {
             const uint32_t idesc_qk = instr_desc(ROWS, KEYS2);
-            const uint32_t idesc_pv = instr_desc(ROWS, p.hd) | (1u << 16);   // B is MN-major
+            const uint32_t idesc_pv = instr_desc(ROWS, p.vd) | (1u << 16);   // B is MN-major
             const int k_steps = p.hd / 16;
             bool ok = mbar_wait(q_full, 0, p.status, 2);
             int done[2] = {0, 0};                      // blocks whose second product a tile has issued
@@ -666,6 +721,7 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 for (int ks = 0; ks < pv_steps; ++ks) {
                     tc_mma_ta(d, pa, db, idesc_pv, keep);
                     keep = 1u;
+                    if (EXTRA) tc_mma_ta(d, pa + KEYS2 / 2, db, idesc_pv, 1u);
                     pa += 8;                               // 16 keys of P: 8 columns
                     db += (uint64_t)(16 * 128 >> 4);       // 16 keys of V
                 }
@@ -734,6 +790,10 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 tc_ld32(tmem_s + 32 * c, part32);
             }
             tc_ld_wait();
+            if (EXTRA) {                                   // scaled and capped here, in place
+#pragma unroll
+                for (int j = 0; j < KEYS2; ++j) raw[j] = __float_as_uint(scaled_capped(p, __uint_as_float(raw[j])));
+            }
             if (need_mask) {
 #pragma unroll
                 for (int j = 0; j < KEYS2; ++j)
@@ -742,7 +802,7 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
             for (int j = 0; j < KEYS2; ++j) mx4[j & 3] = fmaxf(mx4[j & 3], __uint_as_float(raw[j]));
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (EXTRA ? 1.f : p.scale_log2);
             lap(1);
             // The reference maximum moves only when the true one has grown by more than 8; O is rescaled then.  The
             // tile's second product of the block before is done: this block's scores were issued behind it.
@@ -756,7 +816,7 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 if (count > 0) {
 #pragma unroll 1
                     for (int c = 0; c < 8; ++c) {
-                        if (c * 16 < p.hd) {
+                        if (c * 16 < p.vd) {
                             uint32_t o16[16];
                             tc_ld16(tmem_o + c * 16, o16);
                             tc_ld_wait();
@@ -772,6 +832,15 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const float neg_m = m_run == -INFINITY ? 0.f : -m_run;
             float sum4[4] = {0.f, 0.f, 0.f, 0.f};
             // P (bf16, two to a column) goes over the first 64 columns of S.
+            if (EXTRA) {
+#pragma unroll
+                for (int h = 0; h < 4; ++h) {
+                    uint32_t head16[16], rest16[16];
+                    split_weights(&raw[32 * h], neg_m, sum4, head16, rest16);
+                    tc_st16(tmem_s + 16 * h, head16);
+                    tc_st16(tmem_s + KEYS2 / 2 + 16 * h, rest16);
+                }
+            } else
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 uint32_t packed[32];
@@ -793,7 +862,7 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 const int key = j0 + r;
                 if (key > pos_hi_u) {
                     if (!(ok = mbar_wait(v_full + 8 * b, par, p.status, 7))) break;
-                    for (int s = 0; s < slices; ++s) {
+                    for (int s = 0; s < vslices; ++s) {
                         uint4* line = (uint4*)(s_v + b * KV_STAGE2 + s * KSLICE2 + r * 128);
 #pragma unroll
                         for (int q = 0; q < 8; ++q) line[q] = make_uint4(0u, 0u, 0u, 0u);
@@ -811,18 +880,18 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             tc_fence_after();
             lap(4);
             if (ok) {
-                const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-                bf16* dst = p.out + ((size_t)(q_start + t0[x] + t) * p.nq + (size_t)kvh * G + g) * p.hd;
+                const float inv = !valid ? 0.f : EXTRA ? row_factor(p, l_run, m_run, q_start + t0[x] + t, kvh * G + g) : l_run > 0.f ? 1.f / l_run : 0.f;
+                bf16* dst = p.out + ((size_t)(q_start + t0[x] + t) * p.nq + (size_t)kvh * G + g) * p.vd;
 #pragma unroll 1
                 for (int c = 0; c < 4; ++c) {
-                    if (c * 32 < p.hd) {                               // uniform: the load is warp-wide
+                    if (c * 32 < p.vd) {                               // uniform: the load is warp-wide
                         uint32_t o32[32];
                         tc_ld32(tmem_o + c * 32, o32);
                         tc_ld_wait();
                         if (valid) {
 #pragma unroll
                             for (int q = 0; q < 4; ++q) {
-                                if (c * 32 + q * 8 < p.hd) {
+                                if (c * 32 + q * 8 < p.vd) {
                                     float v[8];
 #pragma unroll
                                     for (int j = 0; j < 8; ++j) v[j] = __uint_as_float(o32[q * 8 + j]) * inv;
@@ -904,6 +973,66 @@ FR_EXPORT int attention_tc_supports(int hd, int page, int nq, int nkv, int q_str
            q_stride % 8 == 0;
 }
 
+namespace {
+template <bool EXTRA>
+int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, TcArgs& p, int max_q_len, cudaStream_t stream) {
+    const int T = ROWS / (p.nq / p.nkv);
+    static bool configured = false;
+    if (!configured) {
+        FR_CUDA(cudaFuncSetAttribute(attention_tc_kernel<EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
+        FR_CUDA(cudaFuncSetAttribute(attention_tc_pair_kernel<EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES2));
+        configured = true;
+    }
+    const long long tiles_seq = (max_q_len + T - 1) / T;
+    const long long tiles = tiles_seq * p.nkv * p.n_seqs;
+    if (tiles > 0x7fffffffLL) FR_REFUSE("attention_tc: %lld tiles exceed the grid", tiles);
+    if (tiles_seq >= 2 && use_pairs()) {
+        const dim3 grid((unsigned)(((tiles_seq + 1) / 2) * p.nkv * p.n_seqs));
+        FR_CUDA(fr_launch(attention_tc_pair_kernel<EXTRA>, grid, dim3(THREADS2), SMEM_BYTES2, stream, mq, mk, mv, p));
+        FR_CHECK_LAUNCH("attention_tc (two tiles per CTA)");
+        return FR_OK;
+    }
+    FR_CUDA(fr_launch(attention_tc_kernel<EXTRA>, dim3((unsigned)tiles), dim3(THREADS), SMEM_BYTES, stream, mq, mk, mv, p));
+    FR_CHECK_LAUNCH("attention_tc");
+    return FR_OK;
+}
+
+// checks, tensor maps and what both forms share
+int prepare(TcArgs& p, CUtensorMap& mq, CUtensorMap& mk, CUtensorMap& mv, const void* q, int q_stride, int total_rows, void* out,
+            const void* k_pool, const void* v_pool, int pool_pages, const int* block_table, int table_width, const int* seq_start,
+            const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int nq, int nkv, int hd, int vd, int window, float scale,
+            int* status) {
+    if (!attention_tc_supports(hd, PAGE, nq, nkv, q_stride) || !attention_tc_supports(vd, PAGE, nq, nkv, q_stride))
+        FR_REFUSE("attention_tc: head sizes %d and %d, %d heads on %d kv heads, row stride %d: not for this kernel", hd, vd, nq, nkv, q_stride);
+    if (((uintptr_t)q & 15) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15) || ((uintptr_t)out & 15))
+        FR_REFUSE("attention_tc: buffers must be 16-byte aligned");
+    if (status == nullptr) FR_REFUSE("attention_tc: a status word is needed");
+    const int G = nq / nkv, T = ROWS / G;
+    {
+        const cuuint64_t dims[4] = {(cuuint64_t)hd, (cuuint64_t)G, (cuuint64_t)nkv, (cuuint64_t)total_rows};
+        const cuuint64_t strides[3] = {(cuuint64_t)hd * 2, (cuuint64_t)G * hd * 2, (cuuint64_t)q_stride * 2};
+        const cuuint32_t box[4] = {64, (cuuint32_t)G, 1, (cuuint32_t)T};
+        const int rc = encode(&mq, q, 4, dims, strides, box, "the queries");
+        if (rc) return rc;
+    }
+    for (int which = 0; which < 2; ++which) {
+        const int d = which ? vd : hd;
+        const cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)nkv, (cuuint64_t)pool_pages * PAGE};
+        const cuuint64_t strides[2] = {(cuuint64_t)d * 2, (cuuint64_t)nkv * d * 2};
+        const cuuint32_t box[3] = {64, 1, PAGE};
+        const int rc = encode(which ? &mv : &mk, which ? v_pool : k_pool, 3, dims, strides, box, which ? "the values" : "the keys");
+        if (rc) return rc;
+    }
+    p = TcArgs{};
+    p.out = (bf16*)out; p.block_table = block_table; p.seq_start = seq_start; p.seq_qlen = seq_qlen;
+    p.seq_pos0 = seq_pos0; p.seq_live = seq_live; p.status = status; p.table_width = table_width; p.nq = nq;
+    p.nkv = nkv; p.hd = hd; p.vd = vd; p.window = window; p.pool_rows = pool_pages * PAGE; p.scale_log2 = scale * LOG2E;
+    p.n_seqs = n_seqs;
+    p.trace = attention_tc_trace;
+    return FR_OK;
+}
+}  // namespace
+
 // q: rows of q_stride bf16 (head h at h * hd), total_rows of them; out [rows][nq * hd]; pools [pool_pages][64][nkv][hd]
 // bf16.  seq_start / seq_qlen / seq_pos0: per sequence, its first row, its rows in this step, the position of its
 // first row; seq_live (may be null): indexed by a sequence's first row, negative marks an ended sequence, whose rows
@@ -913,56 +1042,30 @@ FR_EXPORT int attention_tc(const void* q, int q_stride, int total_rows, void* ou
                            const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int max_q_len,
                            int nq, int nkv, int hd, int window, float scale, int* status, cudaStream_t stream) {
     if (n_seqs <= 0 || total_rows <= 0 || max_q_len <= 0) return FR_OK;
-    if (!attention_tc_supports(hd, PAGE, nq, nkv, q_stride))
-        FR_REFUSE("attention_tc: head size %d, %d heads on %d kv heads, row stride %d: not for this kernel", hd, nq, nkv, q_stride);
-    if (((uintptr_t)q & 15) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15) || ((uintptr_t)out & 15))
-        FR_REFUSE("attention_tc: buffers must be 16-byte aligned");
-    if (status == nullptr) FR_REFUSE("attention_tc: a status word is needed");
-    const int G = nq / nkv, T = ROWS / G;
-    CUtensorMap mq, mk, mv;
-    {
-        const cuuint64_t dims[4] = {(cuuint64_t)hd, (cuuint64_t)G, (cuuint64_t)nkv, (cuuint64_t)total_rows};
-        const cuuint64_t strides[3] = {(cuuint64_t)hd * 2, (cuuint64_t)G * hd * 2, (cuuint64_t)q_stride * 2};
-        const cuuint32_t box[4] = {64, (cuuint32_t)G, 1, (cuuint32_t)T};
-        const int rc = encode(&mq, q, 4, dims, strides, box, "the queries");
-        if (rc) return rc;
-    }
-    {
-        const cuuint64_t dims[3] = {(cuuint64_t)hd, (cuuint64_t)nkv, (cuuint64_t)pool_pages * PAGE};
-        const cuuint64_t strides[2] = {(cuuint64_t)hd * 2, (cuuint64_t)nkv * hd * 2};
-        const cuuint32_t box[3] = {64, 1, PAGE};
-        int rc = encode(&mk, k_pool, 3, dims, strides, box, "the keys");
-        if (rc) return rc;
-        rc = encode(&mv, v_pool, 3, dims, strides, box, "the values");
-        if (rc) return rc;
-    }
     TcArgs p;
-    p.out = (bf16*)out; p.block_table = block_table; p.seq_start = seq_start; p.seq_qlen = seq_qlen;
-    p.seq_pos0 = seq_pos0; p.seq_live = seq_live; p.status = status; p.table_width = table_width; p.nq = nq;
-    p.nkv = nkv; p.hd = hd; p.window = window; p.pool_rows = pool_pages * PAGE; p.scale_log2 = scale * LOG2E;
-    p.trace = attention_tc_trace;
-    static bool configured = false;
-    if (!configured) {
-        FR_CUDA(cudaFuncSetAttribute(attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
-        configured = true;
-    }
-    const long long tiles_seq = (max_q_len + T - 1) / T;
-    const long long tiles = tiles_seq * nkv * n_seqs;
-    if (tiles > 0x7fffffffLL) FR_REFUSE("attention_tc: %lld tiles exceed the grid", tiles);
-    p.n_seqs = n_seqs;
-    if (tiles_seq >= 2 && use_pairs()) {
-        static bool configured2 = false;
-        if (!configured2) {
-            FR_CUDA(cudaFuncSetAttribute(attention_tc_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES2));
-            configured2 = true;
-        }
-        const dim3 grid((unsigned)(((tiles_seq + 1) / 2) * nkv * n_seqs));
-        FR_CUDA(fr_launch(attention_tc_pair_kernel, grid, dim3(THREADS2), SMEM_BYTES2, stream, mq, mk, mv, p));
-        FR_CHECK_LAUNCH("attention_tc (two tiles per CTA)");
-        return FR_OK;
-    }
-    const dim3 grid((unsigned)tiles);
-    FR_CUDA(fr_launch(attention_tc_kernel, grid, dim3(THREADS), SMEM_BYTES, stream, mq, mk, mv, p));
-    FR_CHECK_LAUNCH("attention_tc");
-    return FR_OK;
+    CUtensorMap mq, mk, mv;
+    const int rc = prepare(p, mq, mk, mv, q, q_stride, total_rows, out, k_pool, v_pool, pool_pages, block_table, table_width, seq_start, seq_qlen,
+                           seq_pos0, seq_live, n_seqs, nq, nkv, hd, hd, window, scale, status);
+    return rc ? rc : launch<false>(mq, mk, mv, p, max_q_len, stream);
+}
+
+// The form with more to its softmax: values of vd numbers (out [rows][nq * vd], value pool [pool_pages][64][nkv][vd]), softcap (0:
+// none), sink [nq] of sink_dtype (null: none), gate: head h's gate of row r at gate[r * gate_ld + h], bf16 (null: none).
+FR_EXPORT int attention_tc_extra(const void* q, int q_stride, int total_rows, void* out, const void* k_pool, const void* v_pool,
+                                 int pool_pages, const int* block_table, int table_width, const int* seq_start,
+                                 const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int max_q_len,
+                                 int nq, int nkv, int hd, int vd, int window, float scale, float softcap, const void* sink, int sink_dtype,
+                                 const void* gate, int gate_ld, int* status, cudaStream_t stream) {
+    if (n_seqs <= 0 || total_rows <= 0 || max_q_len <= 0) return FR_OK;
+    TcArgs p;
+    CUtensorMap mq, mk, mv;
+    const int rc = prepare(p, mq, mk, mv, q, q_stride, total_rows, out, k_pool, v_pool, pool_pages, block_table, table_width, seq_start, seq_qlen,
+                           seq_pos0, seq_live, n_seqs, nq, nkv, hd, vd, window, scale, status);
+    if (rc) return rc;
+    p.sink = FrVec{sink, sink_dtype};
+    p.gate = (const bf16*)gate;
+    p.gate_ld = gate_ld;
+    p.cap_log2 = softcap * LOG2E;
+    p.two_over_cap_log2 = softcap > 0.f ? 2.0f * scale * LOG2E / softcap : 0.f;
+    return launch<true>(mq, mk, mv, p, max_q_len, stream);
 }

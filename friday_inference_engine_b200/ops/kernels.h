@@ -180,6 +180,8 @@ struct AttentionTc {
     last_error_fn last_error;
     int (*run)(const void*, int, int, void*, const void*, const void*, int, const int*, int, const int*, const int*,
                const int*, const int*, int, int, int, int, int, int, float, int*, cudaStream_t);
+    int (*extra)(const void*, int, int, void*, const void*, const void*, int, const int*, int, const int*, const int*, const int*, const int*, int,
+                 int, int, int, int, int, int, float, float, const void*, int, const void*, int, int*, cudaStream_t);
 };
 struct Sampling {
     last_error_fn last_error;

@@ -564,6 +564,21 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
     const float* pv = pooled ? (const float*)pooled->v_pool : nullptr;
     const int* ptable = pooled ? pooled->block_table : nullptr;
     const int pwidth = pooled ? pooled->table_width : 0;
+    // prompts without window blocks, query multipliers or values that are the keys, in sizes that the tcgen05 kernel takes;
+    // FRIDAY_POOLED_TCGEN05=0 leaves them to the kernel below
+    const bool tcgen05 = proj.dtype == DType::BF16 && !ctx.decode && ctx.max_q_len >= 16 && s.pool == 0 && s.temp_every == 0 && s.v_off >= 0 &&
+                         attn_tc_ && env_on("FRIDAY_POOLED_TCGEN05") && s.dim % 16 == 0 && s.dim <= 128 && s.vdim % 16 == 0 && s.vdim <= 128 &&
+                         tokens.page_size == 64 && s.heads / s.kv_heads <= 128 && proj.ld % 8 == 0 && s.q_off % 8 == 0 && aligned16(proj.data);
+    if (tcgen05) {
+        const auto& a = kernels::attention_tc();
+        Timed t(*this, Attention);
+        call(launches_, a, a.extra((const char*)proj.data + (size_t)s.q_off * dtype_size(proj.dtype), (int)proj.ld, (int)proj.rows(), out.data, tokens.k_pool,
+                                   tokens.v_pool, tokens.pool_pages, tokens.block_table, tokens.table_width, ctx.seq_start, ctx.seq_qlen, ctx.seq_pos0,
+                                   ctx.row_seq, ctx.n_seqs, ctx.max_q_len, s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.scale, s.softcap,
+                                   s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, (int)proj.ld, (int*)status_.get(), stream_),
+             "attention_tc_extra");
+        return out;
+    }
     const bool tc = proj.dtype == DType::BF16 && !ctx.decode && ctx.max_q_len >= 16 && env_on("FRIDAY_POOLED_TC") &&
                     k.prompt_fits(s.dim, s.vdim, tokens.page_size) && ctx.n_seqs <= 65535;
     Timed t(*this, Attention);
