@@ -28,6 +28,9 @@
 //       keys; warps merge through shared memory; the splits of a tile form a thread-block
 //       cluster and merge through each other's shared memory (more than 8 splits: through
 //       a scratch buffer, the last CTA to arrive merging).
+// One-token steps exist in a second form (EXTRA): scores capped as c tanh(s / c), a number per head whose exponential joins the
+// denominator, a sigmoid gate per row and head on the result, and weights that enter the second product as two bf16 numbers each
+// (head and remainder), which keeps them 32-bit in effect.
 // Head sizes: multiples of 16 up to 128.  Others are served by the CUDA-core kernel.
 #include <math.h>
 
@@ -64,7 +67,20 @@ struct MmaArgs {
     int pool_rows;            // rows of a pool (pages x 64): a load from there on is filled with zeros
     int* status;              // a word that receives a code when a bounded wait of the one-token kernel gave up
     unsigned long long* trace;  // for measurements (may be null): [cta][8] timestamps of a one-token step's CTAs
+    // EXTRA only
+    FrVec sink;               // [nq]; p null: none
+    const bf16* gate;         // head h's gate of row r at gate[r * q_stride + h]; null: none
+    float cap_log2, two_over_cap_log2;   // cap (0: none) and, times the scale, 2 / cap, both in units of log2
 };
+
+// one over a row's sum (taken against the maximum big_log2, in units of log2), with the sink and the gate
+template <bool EXTRA>
+__device__ __forceinline__ float row_factor(const MmaArgs& p, float l, float big_log2, int row, int head) {
+    if (EXTRA && p.sink.p != nullptr) l += exp2f(fmaf(p.sink.at(head), LOG2E, -big_log2));
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (EXTRA && p.gate != nullptr) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)row * p.q_stride + head]));
+    return inv;
+}
 
 __device__ __forceinline__ void mark(const MmaArgs& p, int point) {
     if (p.trace != nullptr && threadIdx.x == 0) {
@@ -112,7 +128,7 @@ __device__ __forceinline__ void tma_page(uint32_t dst, const CUtensorMap* map, i
         : "memory");
 }
 
-template <int HD, bool KEYS_MODE>
+template <int HD, bool KEYS_MODE, bool EXTRA>
 __global__ void __launch_bounds__(KEYS_MODE ? (WARPS + 1) * 32 : WARPS * 32)
 attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const MmaArgs p) {
     constexpr int ROW_BYTES = HD * 2 + 16;            // padded: 8 consecutive rows hit 8 different bank groups
@@ -357,7 +373,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
         for (int n = 0; n < NT; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                float v = s[n][e] * p.scale_log2;
+                float v = EXTRA ? fr_capped_log2(s[n][e], p.scale_log2, p.cap_log2, p.two_over_cap_log2) : s[n][e] * p.scale_log2;
                 if (need_mask) {
                     const int j = j0 + n * 8 + 2 * (lane & 3) + (e & 1);
                     if (j > pos_r[e >> 1] || j < lo_r[e >> 1]) v = -INFINITY;
@@ -402,6 +418,15 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
             a[1] = pack_bf16(s[2 * kk][2], s[2 * kk][3]);
             a[2] = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
             a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
+            uint32_t rest[4];                              // what rounding left of the weights
+            if (EXTRA) {
+#pragma unroll
+                for (int w = 0; w < 4; ++w) {
+                    const float (&pair)[4] = s[2 * kk + (w >> 1)];
+                    const int e = 2 * (w & 1);
+                    rest[w] = pack_bf16(pair[e] - __uint_as_float(a[w] << 16), pair[e + 1] - __uint_as_float(a[w] & 0xffff0000u));
+                }
+            }
 #pragma unroll
             for (int dp = 0; dp < DT / 2; ++dp) {
                 uint32_t b[4];
@@ -410,6 +435,10 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
                                      : v_addr + vrow * ROW_BYTES + vch * 16);
                 mma16816(o[2 * dp], a, b[0], b[1]);
                 mma16816(o[2 * dp + 1], a, b[2], b[3]);
+                if (EXTRA) {
+                    mma16816(o[2 * dp], rest, b[0], b[1]);
+                    mma16816(o[2 * dp + 1], rest, b[2], b[3]);
+                }
             }
         }
         if (KEYS_MODE) {
@@ -498,7 +527,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
             }
             const int t = rr / G, h = kvh * G + (rr - t * G);
             const size_t item = (size_t)(q_start + t) * p.nq + h;
-            const float inv = l > 0.f ? 1.f / l : 0.f;
+            const float inv = p.splits == 1 ? row_factor<EXTRA>(p, l, big, q_start + t, h) : 0.f;
             // A row's eight threads take HD / 8 consecutive dimensions each, in pieces of four (two for head sizes
             // that are no multiple of 32): all loads of a piece's four warps are issued before the first is used (one
             // dimension at a time, this loop took 1.6 us of a 9 us kernel).
@@ -584,7 +613,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
                 }
                 const int t = rr2 / G, h = kvh * G + (rr2 - t * G);
                 const size_t item = (size_t)(q_start + t) * p.nq + h;
-                const float inv = l > 0.f ? 1.f / l : 0.f;
+                const float inv = row_factor<EXTRA>(p, l, big, q_start + t, h);
                 uint2 packed;
                 packed.x = pack_bf16(acc.x * inv, acc.y * inv);
                 packed.y = pack_bf16(acc.z * inv, acc.w * inv);
@@ -644,7 +673,10 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
                         }
 #pragma unroll
                     for (int o2 = 1; o2 < 8; o2 <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o2);
-                    if (valid && (tid & 7) == 0) s_inv[r] = l > 0.f ? 1.f / l : 0.f;
+                    if (valid && (tid & 7) == 0) {
+                        const int rr2 = r0 + r, t2 = rr2 / G;
+                        s_inv[r] = row_factor<EXTRA>(p, l, big * LOG2E, q_start + t2, kvh * G + (rr2 - t2 * G));
+                    }
                 }
                 __syncthreads();
                 constexpr int MPIECES = HD / 2;                      // float2 pieces of a row
@@ -740,15 +772,15 @@ constexpr int smem_bytes() {
     return (KEYS_MODE ? 1024 : 0) + ROWS_CTA * ROW_BYTES + (kv > merge ? kv : merge);
 }
 
-template <int HD, bool KEYS_MODE>
+template <int HD, bool KEYS_MODE, bool EXTRA>
 int launch(const CUtensorMap& mk, const CUtensorMap& mv, const MmaArgs& p, dim3 grid, cudaStream_t stream) {
     constexpr int smem = smem_bytes<HD, KEYS_MODE>();
     static bool configured = false;
     if (!configured) {
-        FR_CUDA(cudaFuncSetAttribute(attention_mma_kernel<HD, KEYS_MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        FR_CUDA(cudaFuncSetAttribute(attention_mma_kernel<HD, KEYS_MODE, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         configured = true;
     }
-    FR_CUDA(fr_launch_cluster(attention_mma_kernel<HD, KEYS_MODE>, grid, dim3(KEYS_MODE ? (WARPS + 1) * 32 : WARPS * 32), smem,
+    FR_CUDA(fr_launch_cluster(attention_mma_kernel<HD, KEYS_MODE, EXTRA>, grid, dim3(KEYS_MODE ? (WARPS + 1) * 32 : WARPS * 32), smem,
                               stream, p.cluster ? (unsigned)p.splits : 1u, mk, mv, p));
     FR_CHECK_LAUNCH("attention_mma");
     return FR_OK;
@@ -762,7 +794,7 @@ int clusters_at_once(int size) {
     if (known[size] < 0) {
         known[size] = 0;
         constexpr int smem = smem_bytes<HD, true>();
-        if (cudaFuncSetAttribute(attention_mma_kernel<HD, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) == cudaSuccess) {
+        if (cudaFuncSetAttribute(attention_mma_kernel<HD, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) == cudaSuccess) {
             cudaLaunchConfig_t cfg = {};
             cfg.gridDim = dim3(size * 64);
             cfg.blockDim = dim3((WARPS + 1) * 32);
@@ -775,24 +807,24 @@ int clusters_at_once(int size) {
             cfg.attrs = attr;
             cfg.numAttrs = 1;
             int n = 0;
-            if (cudaOccupancyMaxActiveClusters(&n, attention_mma_kernel<HD, true>, &cfg) == cudaSuccess) known[size] = n;
+            if (cudaOccupancyMaxActiveClusters(&n, attention_mma_kernel<HD, true, false>, &cfg) == cudaSuccess) known[size] = n;
         }
         cudaGetLastError();
     }
     return known[size];
 }
 
-template <bool KEYS_MODE>
+template <bool KEYS_MODE, bool EXTRA>
 int launch_hd(int hd, const CUtensorMap& mk, const CUtensorMap& mv, const MmaArgs& p, dim3 grid, cudaStream_t stream) {
     switch (hd) {
-        case 16: return launch<16, KEYS_MODE>(mk, mv, p, grid, stream);
-        case 32: return launch<32, KEYS_MODE>(mk, mv, p, grid, stream);
-        case 48: return launch<48, KEYS_MODE>(mk, mv, p, grid, stream);
-        case 64: return launch<64, KEYS_MODE>(mk, mv, p, grid, stream);
-        case 80: return launch<80, KEYS_MODE>(mk, mv, p, grid, stream);
-        case 96: return launch<96, KEYS_MODE>(mk, mv, p, grid, stream);
-        case 112: return launch<112, KEYS_MODE>(mk, mv, p, grid, stream);
-        case 128: return launch<128, KEYS_MODE>(mk, mv, p, grid, stream);
+        case 16: return launch<16, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
+        case 32: return launch<32, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
+        case 48: return launch<48, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
+        case 64: return launch<64, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
+        case 80: return launch<80, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
+        case 96: return launch<96, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
+        case 112: return launch<112, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
+        case 128: return launch<128, KEYS_MODE, EXTRA>(mk, mv, p, grid, stream);
         default: FR_REFUSE("attention_mma: head size %d is not built (multiples of 16 up to 128)", hd);
     }
 }
@@ -857,11 +889,11 @@ FR_EXPORT int attention_mma_supports(int hd, int page) { return hd % 16 == 0 && 
 // scratch of rows * nq * splits * (hd + 2) floats.  counters (may be null): n_counters zeroed ints; with them the
 // splits of a one-token step are merged inside the kernel, without them by a second kernel.  status: a device word
 // that receives a code (21 the copying warp, 22 a computing warp) if a bounded wait of a one-token step gives up.
-FR_EXPORT int attention_mma(const void* q, int q_stride, void* out, const void* k_pool, const void* v_pool, int pool_pages,
+static int attention_mma_run(const void* q, int q_stride, void* out, const void* k_pool, const void* v_pool, int pool_pages,
                             const int* block_table, int table_width, int page, const int* seq_start,
                             const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int rows,
                             int max_q_len, int nq, int nkv, int hd, int window, float scale, int keys_mode, int splits,
-                            float* scratch, int* counters, int n_counters, int* status, cudaStream_t stream) {
+                            float* scratch, int* counters, int n_counters, int* status, const MmaArgs* extra, cudaStream_t stream) {
     if (n_seqs <= 0 || rows <= 0) return FR_OK;
     if (!attention_mma_supports(hd, page)) FR_REFUSE("attention_mma: head size %d / page %d is not built", hd, page);
     if (nkv <= 0 || nq % nkv != 0) FR_REFUSE("attention: %d heads cannot share %d key/value heads", nq, nkv);
@@ -869,7 +901,7 @@ FR_EXPORT int attention_mma(const void* q, int q_stride, void* out, const void* 
     if (splits > 8 && scratch == nullptr) FR_REFUSE("attention_mma: more than 8 splits need a scratch buffer");
     if (keys_mode && status == nullptr) FR_REFUSE("attention_mma: one-token steps need a status word");
     if (n_seqs > 65535 || nkv > 65535) FR_REFUSE("attention_mma: %d sequences x %d kv heads exceed the grid", n_seqs, nkv);
-    MmaArgs p;
+    MmaArgs p = extra != nullptr ? *extra : MmaArgs{};
     p.q = (const bf16*)q; p.out = (bf16*)out; p.k_pool = (const bf16*)k_pool; p.v_pool = (const bf16*)v_pool;
     p.block_table = block_table; p.seq_start = seq_start; p.seq_qlen = seq_qlen; p.seq_pos0 = seq_pos0;
     p.seq_live = seq_live; p.part = scratch; p.counters = keys_mode ? counters : nullptr;
@@ -884,6 +916,8 @@ FR_EXPORT int attention_mma(const void* q, int q_stride, void* out, const void* 
     const int tiles = (max_q_len * G + rows_cta - 1) / rows_cta;
     if (p.counters != nullptr && ((long long)n_seqs * nkv * tiles > n_counters || splits > 64))
         p.counters = nullptr;                          // the merge kernel instead
+    if (extra != nullptr && (!keys_mode || (splits > 1 && !p.cluster && p.counters == nullptr)))
+        FR_REFUSE("attention_mma: the form with more to its softmax runs one-token steps whose splits merge inside the kernel");
     dim3 grid(tiles * splits, nkv, n_seqs);
     CUtensorMap mk = {}, mv = {};
     if (keys_mode) {
@@ -894,7 +928,9 @@ FR_EXPORT int attention_mma(const void* q, int q_stride, void* out, const void* 
         rc_map = pool_map(&mv, v_pool, pool_pages, nkv, hd);
         if (rc_map) return rc_map;
     }
-    int rc = keys_mode ? launch_hd<true>(hd, mk, mv, p, grid, stream) : launch_hd<false>(hd, mk, mv, p, grid, stream);
+    int rc = extra != nullptr ? launch_hd<true, true>(hd, mk, mv, p, grid, stream)
+             : keys_mode      ? launch_hd<true, false>(hd, mk, mv, p, grid, stream)
+                              : launch_hd<false, false>(hd, mk, mv, p, grid, stream);
     if (rc) return rc;
     if (splits > 1 && p.counters == nullptr && !p.cluster) {
         MergeArgs mp{scratch, out, rows, nq, hd, splits};
@@ -902,4 +938,31 @@ FR_EXPORT int attention_mma(const void* q, int q_stride, void* out, const void* 
         FR_CHECK_LAUNCH("attention merge");
     }
     return FR_OK;
+}
+
+FR_EXPORT int attention_mma(const void* q, int q_stride, void* out, const void* k_pool, const void* v_pool, int pool_pages,
+                            const int* block_table, int table_width, int page, const int* seq_start,
+                            const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int rows,
+                            int max_q_len, int nq, int nkv, int hd, int window, float scale, int keys_mode, int splits,
+                            float* scratch, int* counters, int n_counters, int* status, cudaStream_t stream) {
+    return attention_mma_run(q, q_stride, out, k_pool, v_pool, pool_pages, block_table, table_width, page, seq_start, seq_qlen, seq_pos0,
+                             seq_live, n_seqs, rows, max_q_len, nq, nkv, hd, window, scale, keys_mode, splits, scratch, counters, n_counters,
+                             status, nullptr, stream);
+}
+
+// One-token steps with more to their softmax: softcap (0: none), sink [nq] of sink_dtype (null: none), gate: head h's gate of row r
+// at gate[r * q_stride + h], bf16 (null: none).  splits as above, at most 64.
+FR_EXPORT int attention_mma_extra(const void* q, int q_stride, void* out, const void* k_pool, const void* v_pool, int pool_pages,
+                                  const int* block_table, int table_width, int page, const int* seq_start,
+                                  const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int rows, int nq, int nkv, int hd,
+                                  int window, float scale, float softcap, const void* sink, int sink_dtype, const void* gate, int splits,
+                                  float* scratch, int* counters, int n_counters, int* status, cudaStream_t stream) {
+    MmaArgs e{};
+    e.sink = FrVec{sink, sink_dtype};
+    e.gate = (const bf16*)gate;
+    e.cap_log2 = softcap * LOG2E;
+    e.two_over_cap_log2 = softcap > 0.f ? 2.0f * scale * LOG2E / softcap : 0.f;
+    return attention_mma_run(q, q_stride, out, k_pool, v_pool, pool_pages, block_table, table_width, page, seq_start, seq_qlen, seq_pos0,
+                             seq_live, n_seqs, rows, 1, nq, nkv, hd, window, scale, 1, splits, scratch, counters, n_counters, status, &e,
+                             stream);
 }

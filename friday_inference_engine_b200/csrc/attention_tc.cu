@@ -136,13 +136,8 @@ __device__ __forceinline__ float exp2_fast(float x) {
     return y;
 }
 
-// a raw score as the softmax sees it, in units of log2: scaled, and capped if there is a cap
-__device__ __forceinline__ float scaled_capped(const TcArgs& p, float raw) {
-    if (p.cap_log2 <= 0.f) return raw * p.scale_log2;
-    float r;
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(exp2_fast(raw * p.two_over_cap_log2) + 1.0f));
-    return fmaf(-2.0f * p.cap_log2, r, p.cap_log2);
-}
+// a raw score as the softmax sees it, in units of log2
+__device__ __forceinline__ float scaled_capped(const TcArgs& p, float raw) { return fr_capped_log2(raw, p.scale_log2, p.cap_log2, p.two_over_cap_log2); }
 // what a row's sum must become for the sink and the gate: result = O * factor
 __device__ __forceinline__ float row_factor(const TcArgs& p, float l, float m, int row, int head) {
     if (p.sink.p != nullptr) l += exp2f(fmaf(p.sink.at(head), LOG2E, -m));

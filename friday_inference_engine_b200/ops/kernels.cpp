@@ -141,7 +141,8 @@ FAMILY(AttentionPooled, attention_pooled, "attention_pooled", resolve(h, fam, "a
        resolve(h, fam, "attention_pooled_rows", t.rows); resolve(h, fam, "attention_pooled_prompt_fits", t.prompt_fits);
        resolve(h, fam, "attention_pooled_prompt", t.prompt);)
 FAMILY(AttentionMma, attention_mma, "attention_mma", resolve(h, fam, "attention_mma", t.run);
-       resolve(h, fam, "attention_mma_clusters_at_once", t.clusters_at_once);)
+       resolve(h, fam, "attention_mma_clusters_at_once", t.clusters_at_once);
+       resolve(h, fam, "attention_mma_extra", t.extra);)
 FAMILY(AttentionTc, attention_tc, "attention_tc", resolve(h, fam, "attention_tc", t.run);
        resolve(h, fam, "attention_tc_extra", t.extra);)
 FAMILY(Sampling, sampling, "sampling", resolve(h, fam, "sampling_sample", t.sample);)

@@ -175,6 +175,8 @@ struct AttentionMma {
                const int*, const int*, int, int, int, int, int, int, int, float, int, int, float*, int*, int, int*,
                cudaStream_t);
     int (*clusters_at_once)(int, int);
+    int (*extra)(const void*, int, void*, const void*, const void*, int, const int*, int, int, const int*, const int*, const int*, const int*, int,
+                 int, int, int, int, int, float, float, const void*, int, const void*, int, float*, int*, int, int*, cudaStream_t);
 };
 struct AttentionTc {
     last_error_fn last_error;

@@ -579,6 +579,25 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
              "attention_tc_extra");
         return out;
     }
+    // one-token steps of the same kinds of layer, heads whose values have the keys' size: the kernel that streams pages by TMA and
+    // shares a sequence's keys among CTAs (FRIDAY_POOLED_MMA=0: the CUDA-core kernel)
+    const int64_t counters_needed = (int64_t)ctx.n_seqs * s.kv_heads * ((s.heads / s.kv_heads + 15) / 16);
+    if (proj.dtype == DType::BF16 && ctx.decode && ctx.seq_start != nullptr && s.pool == 0 && s.temp_every == 0 && s.v_off >= 0 && s.vdim == s.dim &&
+        env_on("FRIDAY_POOLED_MMA") && s.dim % 16 == 0 && s.dim <= 128 && tokens.page_size == 64 && proj.ld % 8 == 0 && s.q_off % 8 == 0 &&
+        aligned16(proj.data) && (int)proj.rows() == ctx.n_seqs && counters_needed <= (int64_t)(attn_counters_.bytes() / sizeof(int)) &&
+        s.kv_heads <= 65535 && ctx.n_seqs <= 65535) {
+        const int splits = decode_splits(ctx.n_seqs, s.heads, s.kv_heads, s.dim, ctx.max_kv_len);
+        float* scratch = splits > 1 ? scratch_floats(proj.rows() * s.heads * splits * (s.dim + 2)) : nullptr;
+        const auto& a = kernels::attention_mma();
+        Timed t(*this, Attention);
+        call(launches_, a, a.extra((const char*)proj.data + (size_t)s.q_off * dtype_size(proj.dtype), (int)proj.ld, out.data, tokens.k_pool, tokens.v_pool,
+                                   tokens.pool_pages, tokens.block_table, tokens.table_width, 64, ctx.seq_start, ctx.seq_qlen, ctx.seq_pos0, ctx.row_seq,
+                                   ctx.n_seqs, (int)proj.rows(), s.heads, s.kv_heads, s.dim, s.window, s.scale, s.softcap,
+                                   s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, splits, scratch,
+                                   (int*)attn_counters_.get(), (int)(attn_counters_.bytes() / sizeof(int)), (int*)status_.get(), stream_),
+             "attention_mma_extra");
+        return out;
+    }
     const bool tc = proj.dtype == DType::BF16 && !ctx.decode && ctx.max_q_len >= 16 && env_on("FRIDAY_POOLED_TC") &&
                     k.prompt_fits(s.dim, s.vdim, tokens.page_size) && ctx.n_seqs <= 65535;
     Timed t(*this, Attention);
