@@ -369,11 +369,12 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
         const int j0 = kb * BLOCK_N + key_base;
         const bool need_mask = (j0 + KPW - 1 > w_pos_min) || (p.window > 0 && j0 < w_lo_max);
         float mx[2] = {-INFINITY, -INFINITY};
+        const bool capping = EXTRA && p.cap_log2 > 0.f;
 #pragma unroll
         for (int n = 0; n < NT; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                float v = EXTRA ? fr_capped_log2(s[n][e], p.scale_log2, p.cap_log2, p.two_over_cap_log2) : s[n][e] * p.scale_log2;
+                float v = EXTRA && capping ? fr_capped(s[n][e], p.cap_log2, p.two_over_cap_log2) : s[n][e] * p.scale_log2;
                 if (need_mask) {
                     const int j = j0 + n * 8 + 2 * (lane & 3) + (e & 1);
                     if (j > pos_r[e >> 1] || j < lo_r[e >> 1]) v = -INFINITY;

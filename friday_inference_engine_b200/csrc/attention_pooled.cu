@@ -573,6 +573,8 @@ __global__ void __launch_bounds__(128, 3) prompt_kernel(PromptArgs p) {
     const int* table = p.block_table + (size_t)seq * p.table_width;
     const int* ptable = p.pool_table != nullptr ? p.pool_table + (size_t)seq * p.pool_table_width : nullptr;
     const float inv_pool = p.pool > 0 ? 1.0f / (float)p.pool : 0.f;
+    const bool capping = p.softcap > 0.f;
+    const float two_over_cap = capping ? 2.0f * 1.4426950408889634f / p.softcap : 0.f;
     const int tiles = pooled_tiles + (last_block - first_block + 1);
     for (int it = 0; it < tiles; ++it) {
         const bool pooled = it < pooled_tiles;
@@ -618,7 +620,9 @@ __global__ void __launch_bounds__(128, 3) prompt_kernel(PromptArgs p) {
                 const int j = b * BN + nt * 8 + 2 * t + (e & 1), half = e >> 1;
                 const int pos = my_pos[half];
                 const bool seen = pos <= last_pos && (pooled ? j < my_blocks[half] : (j <= pos && (p.window <= 0 || pos - j < p.window)));
-                s[nt][e] = seen ? capped(s[nt][e] * mult[half], p.softcap) : -INFINITY;
+                float v = s[nt][e] * mult[half];
+                if (capping) v = fr_capped(v, p.softcap, two_over_cap);
+                s[nt][e] = seen ? v : -INFINITY;
                 m_new[half] = fmaxf(m_new[half], s[nt][e]);
             }
         }

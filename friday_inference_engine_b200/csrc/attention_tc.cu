@@ -31,7 +31,7 @@
 // tokens) are launched first.  Every wait on an mbarrier is bounded (two seconds), then a code goes to `status` and
 // all roles leave their loops.
 //
-// Both kernels exist in a second form (EXTRA) for designs whose softmax has more to it: scores capped as c tanh(s / c), a
+// This kernel exists in a second form (EXTRA) for designs whose softmax has more to it: scores capped as c tanh(s / c), a
 // number per head whose exponential joins the denominator, a sigmoid gate per row and head on the result, and weights that stay
 // 32-bit in effect: P enters the second product as two bf16 numbers each, the head over the first half of its S's columns and
 // the remainder over the second half, with one product for each.  c tanh(s / c) = c - 2 c / (e^(2 s / c) + 1) costs one
@@ -136,8 +136,19 @@ __device__ __forceinline__ float exp2_fast(float x) {
     return y;
 }
 
-// a raw score as the softmax sees it, in units of log2
-__device__ __forceinline__ float scaled_capped(const TcArgs& p, float raw) { return fr_capped_log2(raw, p.scale_log2, p.cap_log2, p.two_over_cap_log2); }
+// raw scores as the softmax sees them, in units of log2 (the choice stands outside the loops: inside, every score would wait for its
+// own branch)
+template <int N>
+__device__ __forceinline__ void scale_and_cap(const TcArgs& p, uint32_t (&raw)[N]) {
+    const float scale = p.scale_log2, cap = p.cap_log2, two = p.two_over_cap_log2;
+    if (cap > 0.f) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) raw[j] = __float_as_uint(fr_capped(__uint_as_float(raw[j]), cap, two));
+    } else {
+#pragma unroll
+        for (int j = 0; j < N; ++j) raw[j] = __float_as_uint(__uint_as_float(raw[j]) * scale);
+    }
+}
 // what a row's sum must become for the sink and the gate: result = O * factor
 __device__ __forceinline__ float row_factor(const TcArgs& p, float l, float m, int row, int head) {
     if (p.sink.p != nullptr) l += exp2f(fmaf(p.sink.at(head), LOG2E, -m));
@@ -399,8 +410,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             // a scheduler has few such warps to choose from); the positive scale is applied to the result.
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             if (EXTRA) {                                   // scaled and capped here, in place
-#pragma unroll
-                for (int j = 0; j < KEYS; ++j) raw[j] = __float_as_uint(scaled_capped(p, __uint_as_float(raw[j])));
+                scale_and_cap(p, raw);
             }
             if (need_mask) {
 #pragma unroll
@@ -550,7 +560,6 @@ constexpr int KSLICE2 = KEYS2 * 128;      // a block's keys (or values), 64 dims
 constexpr int KV_STAGE2 = 2 * KSLICE2;
 constexpr int SMEM_BYTES2 = 4 * SLICE + 4 * KV_STAGE2 + 1024 + 256;
 
-template <bool EXTRA>
 __global__ void __launch_bounds__(THREADS2, 1)
 attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const TcArgs p) {
@@ -716,7 +725,6 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 for (int ks = 0; ks < pv_steps; ++ks) {
                     tc_mma_ta(d, pa, db, idesc_pv, keep);
                     keep = 1u;
-                    if (EXTRA) tc_mma_ta(d, pa + KEYS2 / 2, db, idesc_pv, 1u);
                     pa += 8;                               // 16 keys of P: 8 columns
                     db += (uint64_t)(16 * 128 >> 4);       // 16 keys of V
                 }
@@ -785,10 +793,6 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 tc_ld32(tmem_s + 32 * c, part32);
             }
             tc_ld_wait();
-            if (EXTRA) {                                   // scaled and capped here, in place
-#pragma unroll
-                for (int j = 0; j < KEYS2; ++j) raw[j] = __float_as_uint(scaled_capped(p, __uint_as_float(raw[j])));
-            }
             if (need_mask) {
 #pragma unroll
                 for (int j = 0; j < KEYS2; ++j)
@@ -797,7 +801,7 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
             for (int j = 0; j < KEYS2; ++j) mx4[j & 3] = fmaxf(mx4[j & 3], __uint_as_float(raw[j]));
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (EXTRA ? 1.f : p.scale_log2);
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
             lap(1);
             // The reference maximum moves only when the true one has grown by more than 8; O is rescaled then.  The
             // tile's second product of the block before is done: this block's scores were issued behind it.
@@ -827,15 +831,6 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const float neg_m = m_run == -INFINITY ? 0.f : -m_run;
             float sum4[4] = {0.f, 0.f, 0.f, 0.f};
             // P (bf16, two to a column) goes over the first 64 columns of S.
-            if (EXTRA) {
-#pragma unroll
-                for (int h = 0; h < 4; ++h) {
-                    uint32_t head16[16], rest16[16];
-                    split_weights(&raw[32 * h], neg_m, sum4, head16, rest16);
-                    tc_st16(tmem_s + 16 * h, head16);
-                    tc_st16(tmem_s + KEYS2 / 2 + 16 * h, rest16);
-                }
-            } else
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 uint32_t packed[32];
@@ -875,7 +870,7 @@ attention_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             tc_fence_after();
             lap(4);
             if (ok) {
-                const float inv = !valid ? 0.f : EXTRA ? row_factor(p, l_run, m_run, q_start + t0[x] + t, kvh * G + g) : l_run > 0.f ? 1.f / l_run : 0.f;
+                const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
                 bf16* dst = p.out + ((size_t)(q_start + t0[x] + t) * p.nq + (size_t)kvh * G + g) * p.vd;
 #pragma unroll 1
                 for (int c = 0; c < 4; ++c) {
@@ -975,15 +970,17 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     static bool configured = false;
     if (!configured) {
         FR_CUDA(cudaFuncSetAttribute(attention_tc_kernel<EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
-        FR_CUDA(cudaFuncSetAttribute(attention_tc_pair_kernel<EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES2));
+        FR_CUDA(cudaFuncSetAttribute(attention_tc_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES2));
         configured = true;
     }
     const long long tiles_seq = (max_q_len + T - 1) / T;
     const long long tiles = tiles_seq * p.nkv * p.n_seqs;
     if (tiles > 0x7fffffffLL) FR_REFUSE("attention_tc: %lld tiles exceed the grid", tiles);
-    if (tiles_seq >= 2 && use_pairs()) {
+    // (with a cap and split weights the rows need the registers that two tiles of 128 keys take: one tile per CTA and two CTAs per
+    // SM ran a prompt of 2,048 tokens in 67 us where two tiles per CTA, spilling, took 96)
+    if (!EXTRA && tiles_seq >= 2 && use_pairs()) {
         const dim3 grid((unsigned)(((tiles_seq + 1) / 2) * p.nkv * p.n_seqs));
-        FR_CUDA(fr_launch(attention_tc_pair_kernel<EXTRA>, grid, dim3(THREADS2), SMEM_BYTES2, stream, mq, mk, mv, p));
+        FR_CUDA(fr_launch(attention_tc_pair_kernel, grid, dim3(THREADS2), SMEM_BYTES2, stream, mq, mk, mv, p));
         FR_CHECK_LAUNCH("attention_tc (two tiles per CTA)");
         return FR_OK;
     }

@@ -85,14 +85,14 @@ __device__ __forceinline__ float fr_gated(int kind, float g, float u, float limi
     return g / (1.0f + expf(-g)) * u;
 }
 
-// A raw score as a softmax on powers of two sees it: times scale_log2 or, with a cap c, c tanh(s / c) in the same units, formed as
-// c - 2 c / (e^(2 s / c) + 1); its absolute error is a few units in the last place of c, like the score's own.
-__device__ __forceinline__ float fr_capped_log2(float raw, float scale_log2, float cap_log2, float two_over_cap_log2) {
-    if (cap_log2 <= 0.f) return raw * scale_log2;
+// A raw score capped, cap tanh(scale raw / cap), in any unit (the cap's; natural or log2): two_over_cap is 2 scale / cap times
+// log2(e) in natural units.  Formed as cap - 2 cap / (e^(2 s / cap) + 1): one exponential and one reciprocal; the absolute error is
+// a few units in the last place of the cap, like that of the score itself.
+__device__ __forceinline__ float fr_capped(float raw, float cap, float two_over_cap) {
     float e, r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * two_over_cap_log2));
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * two_over_cap));
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.0f));
-    return fmaf(-2.0f * cap_log2, r, cap_log2);
+    return fmaf(-2.0f * cap, r, cap);
 }
 
 // The rotation of one pair of a rotary encoding, the same instructions wherever it is applied.

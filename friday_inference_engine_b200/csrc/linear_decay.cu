@@ -133,41 +133,61 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
     hi = *(const uint32_t*)&h;
     lo = pack2(x - __bfloat162float(hx), y - __bfloat162float(hy));
 }
-// silu of channels c .. c + 7 of a row of n channels (zero beyond), fp32 values that bf16 holds exactly
-__device__ __forceinline__ void silu8(const bf16* src, int c, int n, float (&v)[8]) {
-    if (c + 8 <= n && (((uintptr_t)(src + c)) & 15) == 0) {
-        const uint4 r = *(const uint4*)(src + c);
-        const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+constexpr int THR = 256;             // threads of a chunk's block
+
+// channels c .. c + 7 of a row of n channels (zero beyond) as stored
+__device__ __forceinline__ uint4 raw8(const bf16* src, int c, int n) {
+    if (c + 8 <= n && (((uintptr_t)(src + c)) & 15) == 0) return *(const uint4*)(src + c);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    bf16* e = (bf16*)&v;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            v[2 * i] = silu_as<bf16>(__uint_as_float(w[i] << 16));
-            v[2 * i + 1] = silu_as<bf16>(__uint_as_float(w[i] & 0xffff0000u));
-        }
-        return;
+    for (int i = 0; i < 8; ++i) e[i] = c + i < n ? src[c + i] : __float2bfloat16_rn(0.f);
+    return v;
+}
+// their silu, fp32 values that bf16 holds exactly
+__device__ __forceinline__ void silu8(const uint4& r, float (&v)[8]) {
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = silu_as<bf16>(__uint_as_float(w[i] << 16));
+        v[2 * i + 1] = silu_as<bf16>(__uint_as_float(w[i] & 0xffff0000u));
     }
-#pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = c + i < n ? silu_as<bf16>(__bfloat162float(src[c + i])) : 0.f;
 }
 __device__ __forceinline__ uint4 pack8(const float (&v)[8]) { return make_uint4(pack2(v[0], v[1]), pack2(v[2], v[3]), pack2(v[4], v[5]), pack2(v[6], v[7])); }
 
-// rows r0 .. r0 + n - 1 of a head's channels into a tile [CH][D + PAD], silu applied, zeros below row n
+// A thread's share of the rows r0 .. r0 + n - 1 of a head's channels: all loads first (`fetch`), used later
+template <int D> constexpr int pieces_of() { return (CH * (D / 8) + THR - 1) / THR; }
 template <int D>
-__device__ __forceinline__ void stage_rows(const DecayArgs& p, int off, int width, int r0, int n, bf16* tile) {
-    for (int idx = threadIdx.x; idx < CH * (D / 8); idx += 128) {
-        const int t = idx / (D / 8), c = (idx % (D / 8)) * 8;
-        float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        if (t < n) silu8((const bf16*)p.proj + (size_t)(r0 + t) * p.ld + off, c, width, v);
+__device__ __forceinline__ void fetch_rows(const DecayArgs& p, int off, int width, int r0, int n, uint4 (&raw)[pieces_of<D>()]) {
+#pragma unroll
+    for (int i = 0; i < pieces_of<D>(); ++i) {
+        const int idx = threadIdx.x + i * THR, t = idx / (D / 8), c = (idx % (D / 8)) * 8;
+        raw[i] = make_uint4(0, 0, 0, 0);
+        if (t < n) raw[i] = raw8((const bf16*)p.proj + (size_t)(r0 + t) * p.ld + off, c, width);
+    }
+}
+// into a tile [CH][D + PAD], silu applied (zero stays zero)
+template <int D>
+__device__ __forceinline__ void put_rows(const uint4 (&raw)[pieces_of<D>()], bf16* tile) {
+#pragma unroll
+    for (int i = 0; i < pieces_of<D>(); ++i) {
+        const int idx = threadIdx.x + i * THR, t = idx / (D / 8), c = (idx % (D / 8)) * 8;
+        if (t >= CH) break;
+        float v[8];
+        silu8(raw[i], v);
         *(uint4*)(tile + t * (D + PAD) + c) = pack8(v);
     }
 }
 
 template <int DK, int DV>
-__global__ void __launch_bounds__(128) chunk_states_kernel(DecayArgs p) {
+__global__ void __launch_bounds__(THR) chunk_states_kernel(DecayArgs p) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* skh = (bf16*)smem_raw;                          // [CH][DK + PAD] scaled keys, head
     bf16* skl = skh + CH * (DK + PAD);                    // and remainder
     bf16* sv = skl + CH * (DK + PAD);                     // [CH][DV + PAD]
-    constexpr int MT = DK / 16, PER = (MT + 3) / 4;       // tiles of 16 key channels, and how many a warp owns
+    __shared__ float pw[CH];
+    // warps share the tiles of 16 key channels; where there are fewer tiles than warps, the value channels as well
+    constexpr int MT = DK / 16, PER = (MT + 7) / 8, COLS = MT >= 8 ? 1 : 8 / MT, DVW = DV / COLS < 16 ? 16 : DV / COLS;
     const int c = blockIdx.x, head = blockIdx.y, seq = blockIdx.z;
     const int qlen = p.seq_qlen[seq];
     if (c * CH >= qlen) return;
@@ -176,47 +196,53 @@ __global__ void __launch_bounds__(128) chunk_states_kernel(DecayArgs p) {
     fr_pdl_wait();
     fr_pdl_launch();
     if (p.row_seq[r0] < 0) return;
-    const float d = p.decay[head];
-    for (int idx = threadIdx.x; idx < CH * (DK / 8); idx += 128) {
-        const int t = idx / (DK / 8), k = (idx % (DK / 8)) * 8;
-        float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        if (t < n) {
-            silu8((const bf16*)p.proj + (size_t)(r0 + t) * p.ld + p.k_off + head * p.dk, k, p.dk, v);
-            const float f = powf(d, (float)(n - 1 - t));
+    uint4 kr[pieces_of<DK>()], vr[pieces_of<DV>()];
+    fetch_rows<DK>(p, p.k_off + head * p.dk, p.dk, r0, n, kr);
+    fetch_rows<DV>(p, p.v_off + head * p.dv, p.dv, r0, n, vr);
+    if (threadIdx.x < CH) pw[threadIdx.x] = powf(p.decay[head], (float)threadIdx.x);
+    __syncthreads();
 #pragma unroll
-            for (int i = 0; i < 8; ++i) v[i] *= f;
-        }
+    for (int i = 0; i < pieces_of<DK>(); ++i) {
+        const int idx = threadIdx.x + i * THR, t = idx / (DK / 8), k = (idx % (DK / 8)) * 8;
+        if (t >= CH) break;
+        float v[8];
+        silu8(kr[i], v);
+        const float f = t < n ? pw[n - 1 - t] : 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= f;
         uint4 hi, lo;
         split2(v[0], v[1], hi.x, lo.x); split2(v[2], v[3], hi.y, lo.y); split2(v[4], v[5], hi.z, lo.z); split2(v[6], v[7], hi.w, lo.w);
         *(uint4*)(skh + t * (DK + PAD) + k) = hi;
         *(uint4*)(skl + t * (DK + PAD) + k) = lo;
     }
-    stage_rows<DV>(p, p.v_off + head * p.dv, p.dv, r0, n, sv);
+    put_rows<DV>(vr, sv);
     __syncthreads();
-    float acc[PER][DV / 8][4];
+    const int m0 = COLS == 1 ? warp : warp % MT, v0 = COLS == 1 ? 0 : (warp / MT) * DVW;
+    if (v0 >= DV) return;
+    float acc[PER][DVW / 8][4];
 #pragma unroll
     for (int m = 0; m < PER; ++m)
 #pragma unroll
-        for (int j = 0; j < DV / 8; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
+        for (int j = 0; j < DVW / 8; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
     const int a_row = (lane & 7) + ((lane >> 4) & 1) * 8, a_col = ((lane >> 3) & 1) * 8;      // A is stored [token][key channel]
 #pragma unroll
     for (int ks = 0; ks < CH / 16; ++ks) {
         uint32_t ah[PER][4], al[PER][4];
 #pragma unroll
         for (int m = 0; m < PER; ++m) {
-            const int tile = warp + 4 * m;
+            const int tile = m0 + 8 * m;
             if (tile < MT) {
                 ldsm4t(ah[m], skh + (ks * 16 + a_row) * (DK + PAD) + tile * 16 + a_col);
                 ldsm4t(al[m], skl + (ks * 16 + a_row) * (DK + PAD) + tile * 16 + a_col);
             }
         }
 #pragma unroll
-        for (int j = 0; j < DV / 16; ++j) {
+        for (int j = 0; j < DVW / 16; ++j) {
             uint32_t b[4];
-            ldsm4t(b, sv + (ks * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
+            ldsm4t(b, sv + (ks * 16 + (lane & 15)) * (DV + PAD) + v0 + j * 16 + (lane >> 4) * 8);
 #pragma unroll
             for (int m = 0; m < PER; ++m) {
-                if (warp + 4 * m < MT) {
+                if (m0 + 8 * m < MT) {
                     mma_16816(acc[m][2 * j], ah[m], b[0], b[1]);
                     mma_16816(acc[m][2 * j], al[m], b[0], b[1]);
                     mma_16816(acc[m][2 * j + 1], ah[m], b[2], b[3]);
@@ -229,15 +255,15 @@ __global__ void __launch_bounds__(128) chunk_states_kernel(DecayArgs p) {
     const bool pairs = p.dv % 2 == 0;
 #pragma unroll
     for (int m = 0; m < PER; ++m) {
-        const int tile = warp + 4 * m;
+        const int tile = m0 + 8 * m;
         if (tile >= MT) continue;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const int k = tile * 16 + g + 8 * half;
             if (k >= p.dk) continue;
 #pragma unroll
-            for (int j = 0; j < DV / 8; ++j) {
-                const int col = j * 8 + 2 * t4;
+            for (int j = 0; j < DVW / 8; ++j) {
+                const int col = v0 + j * 8 + 2 * t4;
                 float* dst = U + (size_t)k * p.dv + col;
                 if (pairs && col + 1 < p.dv) *(float2*)dst = make_float2(acc[m][j][2 * half], acc[m][j][2 * half + 1]);
                 else {
@@ -292,9 +318,10 @@ constexpr int outputs_smem() {
 }
 
 template <int DK, int DV>
-__global__ void __launch_bounds__(128) chunk_outputs_kernel(DecayArgs p) {
+__global__ void __launch_bounds__(THR) chunk_outputs_kernel(DecayArgs p) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     constexpr int states = 2 * DK * (DV + PAD), rows = CH * (DK + PAD) + CH * (DV + PAD);
+    constexpr int DH = DV / 2;                            // value channels of a warp: two warps share 16 rows
     bf16* sq = (bf16*)smem_raw;                           // [CH][DK + PAD]
     bf16* sh = sq + CH * (DK + PAD);                      // [DK][DV + PAD] the chunk's starting state, head
     bf16* sl = sh + DK * (DV + PAD);                      // and remainder; once they are used, in their place:
@@ -306,79 +333,96 @@ __global__ void __launch_bounds__(128) chunk_outputs_kernel(DecayArgs p) {
     if (c * CH >= qlen) return;
     const int r0 = p.seq_start[seq] + c * CH, n = min(CH, qlen - c * CH);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+    const int w_row = (warp & 3) * 16, v0 = (warp >> 2) * DH;
     fr_pdl_wait();
     fr_pdl_launch();
     if (p.row_seq[r0] < 0) return;
-    const float d = p.decay[head];
-    if (threadIdx.x <= CH) pw[threadIdx.x] = powf(d, (float)threadIdx.x);
-    stage_rows<DK>(p, p.q_off + head * p.dk, p.dk, r0, n, sq);
+    uint4 qr[pieces_of<DK>()];
+    fetch_rows<DK>(p, p.q_off + head * p.dk, p.dk, r0, n, qr);
+    if (threadIdx.x <= CH) pw[threadIdx.x] = powf(p.decay[head], (float)threadIdx.x);
     const float* S = p.chunk + (((size_t)seq * p.max_chunks + c) * p.heads + head) * p.dk * p.dv;
     const bool fours = p.dv % 4 == 0;
-    for (int idx = threadIdx.x; idx < DK * (DV / 4); idx += 128) {
-        const int k = idx / (DV / 4), v = (idx % (DV / 4)) * 4;
-        float x[4] = {0.f, 0.f, 0.f, 0.f};
-        if (k < p.dk) {
-            const float* src = S + (size_t)k * p.dv + v;
-            if (fours && v + 4 <= p.dv) {
-                const float4 f = *(const float4*)src;
-                x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w;
-            } else {
+    constexpr int ITEMS = DK * (DV / 4) / THR, BATCH = ITEMS < 8 ? ITEMS : 8;       // pieces of four numbers; loads in flight
+#pragma unroll 1
+    for (int i0 = 0; i0 < ITEMS; i0 += BATCH) {
+        float4 x[BATCH];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) x[i] = v + i < p.dv ? src[i] : 0.f;
+        for (int i = 0; i < BATCH; ++i) {
+            const int idx = threadIdx.x + (i0 + i) * THR, k = idx / (DV / 4), v = (idx % (DV / 4)) * 4;
+            x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (k >= p.dk || v >= p.dv) continue;
+            const float* src = S + (size_t)k * p.dv + v;
+            if (fours) x[i] = *(const float4*)src;
+            else {
+                x[i].x = src[0];
+                if (v + 1 < p.dv) x[i].y = src[1];
+                if (v + 2 < p.dv) x[i].z = src[2];
+                if (v + 3 < p.dv) x[i].w = src[3];
             }
         }
-        uint2 hi, lo;
-        split2(x[0], x[1], hi.x, lo.x);
-        split2(x[2], x[3], hi.y, lo.y);
-        *(uint2*)(sh + k * (DV + PAD) + v) = hi;
-        *(uint2*)(sl + k * (DV + PAD) + v) = lo;
-    }
-    __syncthreads();
-    // what the state before the chunk gives its rows
-    float o[DV / 8][4];
 #pragma unroll
-    for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-    uint32_t qa[DK / 16][4];
-#pragma unroll
-    for (int ks = 0; ks < DK / 16; ++ks) {
-        ldsm4(qa[ks], sq + (warp * 16 + (lane & 15)) * (DK + PAD) + ks * 16 + (lane >> 4) * 8);
-#pragma unroll
-        for (int j = 0; j < DV / 16; ++j) {
-            uint32_t bh[4], bl[4];
-            ldsm4t(bh, sh + (ks * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
-            ldsm4t(bl, sl + (ks * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
-            mma_16816(o[2 * j], qa[ks], bh[0], bh[1]);
-            mma_16816(o[2 * j], qa[ks], bl[0], bl[1]);
-            mma_16816(o[2 * j + 1], qa[ks], bh[2], bh[3]);
-            mma_16816(o[2 * j + 1], qa[ks], bl[2], bl[3]);
+        for (int i = 0; i < BATCH; ++i) {
+            const int idx = threadIdx.x + (i0 + i) * THR, k = idx / (DV / 4), v = (idx % (DV / 4)) * 4;
+            uint2 hi, lo;
+            split2(x[i].x, x[i].y, hi.x, lo.x);
+            split2(x[i].z, x[i].w, hi.y, lo.y);
+            *(uint2*)(sh + k * (DV + PAD) + v) = hi;
+            *(uint2*)(sl + k * (DV + PAD) + v) = lo;
         }
     }
-    const int row[2] = {warp * 16 + g, warp * 16 + g + 8};
+    put_rows<DK>(qr, sq);
+    __syncthreads();
+    // the chunk's keys and values are on their way while the state is read
+    uint4 kr[pieces_of<DK>()], vr[pieces_of<DV>()];
+    fetch_rows<DK>(p, p.k_off + head * p.dk, p.dk, r0, n, kr);
+    fetch_rows<DV>(p, p.v_off + head * p.dv, p.dv, r0, n, vr);
+    // what the state before the chunk gives its rows
+    float o[DH / 8][4];
+#pragma unroll
+    for (int j = 0; j < DH / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    const bf16* q_at = sq + (w_row + (lane & 15)) * (DK + PAD) + (lane >> 4) * 8;
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks) {
+        uint32_t qa[4];
+        ldsm4(qa, q_at + ks * 16);
+#pragma unroll
+        for (int j = 0; j < DH / 16; ++j) {
+            uint32_t bh[4], bl[4];
+            ldsm4t(bh, sh + (ks * 16 + (lane & 15)) * (DV + PAD) + v0 + j * 16 + (lane >> 4) * 8);
+            ldsm4t(bl, sl + (ks * 16 + (lane & 15)) * (DV + PAD) + v0 + j * 16 + (lane >> 4) * 8);
+            mma_16816(o[2 * j], qa, bh[0], bh[1]);
+            mma_16816(o[2 * j], qa, bl[0], bl[1]);
+            mma_16816(o[2 * j + 1], qa, bh[2], bh[3]);
+            mma_16816(o[2 * j + 1], qa, bl[2], bl[3]);
+        }
+    }
+    const int row[2] = {w_row + g, w_row + g + 8};
     const float f0 = pw[row[0] + 1], f1 = pw[row[1] + 1];
 #pragma unroll
-    for (int j = 0; j < DV / 8; ++j) {
+    for (int j = 0; j < DH / 8; ++j) {
         o[j][0] *= f0;
         o[j][1] *= f0;
         o[j][2] *= f1;
         o[j][3] *= f1;
     }
     __syncthreads();
-    stage_rows<DK>(p, p.k_off + head * p.dk, p.dk, r0, n, sk);
-    stage_rows<DV>(p, p.v_off + head * p.dv, p.dv, r0, n, sv);
+    put_rows<DK>(kr, sk);
+    put_rows<DV>(vr, sv);
     __syncthreads();
     // and the chunk's own tokens, those up to each row (a warp's rows see no token beyond its last row)
 #pragma unroll
     for (int kk = 0; kk < CH / 16; ++kk) {
-        if (kk > warp) break;
+        if (kk > (warp & 3)) break;
         float s[2][4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[0][e] = s[1][e] = 0.f;
 #pragma unroll
         for (int ks = 0; ks < DK / 16; ++ks) {
-            uint32_t b[4];                                // keys kk * 16 .. + 15: B is stored [token][key channel]
+            uint32_t qa[4], b[4];                         // keys kk * 16 .. + 15: B is stored [token][key channel]
+            ldsm4(qa, q_at + ks * 16);
             ldsm4(b, sk + (kk * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * (DK + PAD) + ks * 16 + ((lane >> 3) & 1) * 8);
-            mma_16816(s[0], qa[ks], b[0], b[1]);
-            mma_16816(s[1], qa[ks], b[2], b[3]);
+            mma_16816(s[0], qa, b[0], b[1]);
+            mma_16816(s[1], qa, b[2], b[3]);
         }
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
@@ -393,9 +437,9 @@ __global__ void __launch_bounds__(128) chunk_outputs_kernel(DecayArgs p) {
         split2(s[1][0], s[1][1], hi[2], lo[2]);
         split2(s[1][2], s[1][3], hi[3], lo[3]);
 #pragma unroll
-        for (int j = 0; j < DV / 16; ++j) {
+        for (int j = 0; j < DH / 16; ++j) {
             uint32_t b[4];
-            ldsm4t(b, sv + (kk * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
+            ldsm4t(b, sv + (kk * 16 + (lane & 15)) * (DV + PAD) + v0 + j * 16 + (lane >> 4) * 8);
             mma_16816(o[2 * j], hi, b[0], b[1]);
             mma_16816(o[2 * j], lo, b[0], b[1]);
             mma_16816(o[2 * j + 1], hi, b[2], b[3]);
@@ -408,8 +452,8 @@ __global__ void __launch_bounds__(128) chunk_outputs_kernel(DecayArgs p) {
         if (row[half] >= n) continue;
         float* dst = p.out + (size_t)(r0 + row[half]) * ((size_t)p.heads * p.dv) + (size_t)head * p.dv;
 #pragma unroll
-        for (int j = 0; j < DV / 8; ++j) {
-            const int col = j * 8 + 2 * t4;
+        for (int j = 0; j < DH / 8; ++j) {
+            const int col = v0 + j * 8 + 2 * t4;
             if (pairs && col + 1 < p.dv) *(float2*)(dst + col) = make_float2(o[j][2 * half], o[j][2 * half + 1]);
             else {
                 if (col < p.dv) dst[col] = o[j][2 * half];
@@ -429,13 +473,13 @@ int launch_chunks(const DecayArgs& p, int n_seqs, cudaStream_t stream) {
         set = true;
     }
     const dim3 grid(p.max_chunks, p.heads, n_seqs);
-    FR_CUDA(fr_launch(chunk_states_kernel<DK, DV>, grid, dim3(128), smem_a, stream, p));
+    FR_CUDA(fr_launch(chunk_states_kernel<DK, DV>, grid, dim3(THR), smem_a, stream, p));
     const int per = p.dk * p.dv;
     if (per % 4 == 0 && p.state_stride % 4 == 0 && ((((uintptr_t)p.state) | ((uintptr_t)p.chunk)) & 15) == 0)
         FR_CUDA(fr_launch(chunk_chain_kernel<float4>, dim3(n_seqs, p.heads, (per / 4 + 255) / 256), dim3(256), 0, stream, p));
     else
         FR_CUDA(fr_launch(chunk_chain_kernel<float>, dim3(n_seqs, p.heads, (per + 255) / 256), dim3(256), 0, stream, p));
-    FR_CUDA(fr_launch(chunk_outputs_kernel<DK, DV>, grid, dim3(128), smem_c, stream, p));
+    FR_CUDA(fr_launch(chunk_outputs_kernel<DK, DV>, grid, dim3(THR), smem_c, stream, p));
     FR_CHECK_LAUNCH("linear_decay chunks");
     return FR_OK;
 }

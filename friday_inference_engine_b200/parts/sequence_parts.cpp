@@ -434,9 +434,18 @@ public:
                 Tensor act = ops.linear_swiglu(Rows(x), tensor("w_shared"), act_, shared_limit_, slope_);
                 shared = ops.linear(Rows(act), tensor("shared.down"), nullptr, nullptr, (int)DType::F32);
             }
-            residual = ops.shared_and_self(residual_in.defined() ? &residual_in : nullptr, shared.defined() ? &shared : nullptr,
-                                           shared_gate_.empty() ? nullptr : &logits, (int64_t)experts_ + identity_,
-                                           r.self.defined() ? &r.self : nullptr, x);
+            auto with_shared = [&](const Tensor& to) {
+                return ops.shared_and_self(to.defined() ? &to : nullptr, shared.defined() ? &shared : nullptr, shared_gate_.empty() ? nullptr : &logits,
+                                           (int64_t)experts_ + identity_, r.self.defined() ? &r.self : nullptr, x);
+            };
+            if (dense && !residual_in.defined() && x.rows() > 128) {
+                // many rows and no stream: the chosen experts' sum first, the rest joins it in one kernel (the product's own sum
+                // with 32-bit rows is a kernel of its own for many rows)
+                Tensor act = ops.linear_swiglu(Rows(x), tensor("w_gate_up"), act_, limit_, slope_);
+                ops.scale_by_route(act, r.dense, experts_, inner_);
+                return PartOut(with_shared(ops.linear(Rows(act), tensor("w_down"), nullptr, nullptr, (int)DType::F32)));
+            }
+            residual = with_shared(residual_in);
         }
         if (grouped)
             return PartOut(ops.experts_grouped(x, r, tensor("w_gate_up"), tensor("w_down"), residual, top_, inner_, act_, limit_, slope_));
