@@ -211,9 +211,16 @@ __global__ void __launch_bounds__(WHOLE_THREADS) prepare_whole_kernel(PrepArgs p
             for (int c = threadIdx.x * 8; c < n; c += WHOLE_THREADS * 8) {
                 float v[8];
                 load8(src + c, v);
-                if (w.p != nullptr)
+                if (w.p != nullptr) {
+                    float w0[4], w1[4];
+                    w.four(c, w0);
+                    w.four(c + 4, w1);
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * w.at(c + i);
+                    for (int i = 0; i < 4; ++i) {
+                        v[i] = v[i] * inv * w0[i];
+                        v[4 + i] = v[4 + i] * inv * w1[i];
+                    }
+                }
                 const int d = c % p.dim;
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {

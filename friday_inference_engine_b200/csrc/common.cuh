@@ -71,6 +71,19 @@ struct FrVec {
     __device__ __forceinline__ float at(int i) const {
         return dtype == FR_F32 ? ((const float*)p)[i] : __bfloat162float(((const __nv_bfloat16*)p)[i]);
     }
+    // elements i .. i + 3, i a multiple of four (one load where the vector's start allows it)
+    __device__ __forceinline__ void four(int i, float (&v)[4]) const {
+        if ((((uintptr_t)p) & 15) != 0) {
+            for (int k = 0; k < 4; ++k) v[k] = at(i + k);
+        } else if (dtype == FR_F32) {
+            const float4 a = *(const float4*)((const float*)p + i);
+            v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+        } else {
+            const uint2 r = *(const uint2*)((const __nv_bfloat16*)p + i);
+            v[0] = __uint_as_float(r.x << 16); v[1] = __uint_as_float(r.x & 0xffff0000u);
+            v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
+        }
+    }
 };
 
 // A gated unit: the gate's activation times up.  kind 1: silu; 2: the tanh form of gelu; 3: both clipped, g = min(gate, limit) and

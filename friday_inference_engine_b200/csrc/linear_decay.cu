@@ -535,9 +535,11 @@ __global__ void __launch_bounds__(256) row_norm_gate_kernel(const float* __restr
         for (int c = threadIdx.x * 4; c < n; c += 1024) {
             const float4 v = *(const float4*)(x + c);
             const float xs[4] = {v.x, v.y, v.z, v.w};
-            float r[4];
+            float r[4], ws[4], gs[4];
+            w.four(c, ws);
+            FrVec{g, sizeof(T) == 2 ? FR_BF16 : FR_F32}.four(c, gs);
 #pragma unroll
-            for (int i = 0; i < 4; ++i) r[i] = xs[i] * inv * w.at(c + i) / (1.0f + expf(-fr_load(g + c + i)));
+            for (int i = 0; i < 4; ++i) r[i] = xs[i] * inv * ws[i] / (1.0f + expf(-gs[i]));
             if constexpr (sizeof(T) == 2) *(uint2*)(y + c) = make_uint2(pack2(r[0], r[1]), pack2(r[2], r[3]));
             else *(float4*)(y + c) = make_float4(r[0], r[1], r[2], r[3]);
         }

@@ -637,10 +637,11 @@ post_norm_add_vec_kernel(const float* __restrict__ x, const float* __restrict__ 
         const int i = threadIdx.x + k * 256;
         if (i < n4) {
             const float yv[4] = {v[k].x, v[k].y, v[k].z, v[k].w}, xv[4] = {r[k].x, r[k].y, r[k].z, r[k].w};
-            float o[4];
+            float o[4], wv[4];
+            w.four(4 * i, wv);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                o[e] = fmaf(mult, yv[e] * inv * w.at(4 * i + e), xv[e]);
+                o[e] = fmaf(mult, yv[e] * inv * wv[e], xv[e]);
                 s2 = fmaf(o[e], o[e], s2);
             }
             store4(out + base + 4 * i, o);
@@ -656,9 +657,10 @@ post_norm_add_vec_kernel(const float* __restrict__ x, const float* __restrict__ 
         const int i = threadIdx.x + k * 256;
         if (i < n4) {
             const float ov[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
-            float o[4];
+            float o[4], wv[4];
+            w2.four(4 * i, wv);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) o[e] = ov[e] * inv2 * w2.at(4 * i + e);
+            for (int e = 0; e < 4; ++e) o[e] = ov[e] * inv2 * wv[e];
             store4(next + base + 4 * i, o);
         }
     }

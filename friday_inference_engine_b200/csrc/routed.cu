@@ -769,9 +769,12 @@ shared_and_self_kernel(const float* __restrict__ residual, const float* __restri
                     const float4 s = *(const float4*)(shared + base + c);
                     v[0] = g * s.x; v[1] = g * s.y; v[2] = g * s.z; v[3] = g * s.w;
                 }
-                if (w != 0.f)
+                if (w != 0.f) {
+                    float hs[4];
+                    FrVec{h + base, sizeof(T) == 2 ? FR_BF16 : FR_F32}.four(c, hs);
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) v[i] = fmaf(w, fr_load(h + base + c + i), v[i]);
+                    for (int i = 0; i < 4; ++i) v[i] = fmaf(w, hs[i], v[i]);
+                }
                 if (residual != nullptr) {
                     const float4 r = *(const float4*)(residual + base + c);
                     v[0] += r.x; v[1] += r.y; v[2] += r.z; v[3] += r.w;

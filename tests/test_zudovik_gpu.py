@@ -310,6 +310,22 @@ def test_forms_of_the_experts(root, form, monkeypatch):
     agree(got, root, "R", p, list(range(150)), "bfloat16", "R, experts %s" % form)
 
 
+@pytest.mark.parametrize("splits", ["1", "2", "5", "8", "11"])
+def test_one_token_steps_in_splits(root, splits, monkeypatch):
+    """A sequence's keys shared among CTAs, as a cluster and through memory, some of them with no key at all: caps, sinks and
+    gates join once, whoever merges."""
+    monkeypatch.setenv("FRIDAY_ATTN_SPLITS", splits)
+    eng, cfg, _ = engine(root, "R", "bfloat16")
+    ps = prompts([290, 40], cfg["vocab"], 19)
+    slots = [eng.alloc_slot() for _ in ps]
+    eng.step(slots, [p[:-3] for p in ps], [[], []], to="host")
+    got = [eng.step(slots, [[p[len(p) - 3 + k]] for p in ps], [[0], [0]], to="host") for k in range(3)]
+    for i, p in enumerate(ps):
+        eng.free_slot(slots[i])
+        agree(np.stack([g[i] for g in got]), root, "R", p, list(range(len(p) - 3, len(p))), "bfloat16", "R in %s splits, request %d" % (splits, i))
+    eng.check()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_slots_and_pages_used_again(root, dtype):
     """A slot that held a long request is given to a short one: states start anew, stale pages are not read."""
