@@ -27,7 +27,7 @@ void FreeList::give(int i) {
 
 KVGroup::KVGroup(const CacheRequest& req, const std::vector<int>& ents, int n_slots, int pages_, int width_, DType dt,
                  bool on_device)
-    : request(req), entries(ents), window(req.window), n_pages(pages_), width(width_), dtype(req.store_f32 ? DType::F32 : dt), pages(pages_, "page"),
+    : request(req), entries(ents), window(req.window), chunk(req.chunk), n_pages(pages_), width(width_), dtype(req.store_f32 ? DType::F32 : dt), pages(pages_, "page"),
       table((size_t)n_slots * width_, -1) {
     if (on_device) {
         k_pool = DeviceBuffer(entry_bytes() * entries.size());
@@ -41,10 +41,12 @@ int KVGroup::index_of(int entry) const {
     return -1;
 }
 
-int KVGroup::first_needed_page(int start_pos) const {
-    if (window <= 0) return 0;
-    return std::max(0, start_pos - window + 1) / PAGE;
+int KVGroup::first_key(int pos) const {
+    if (chunk > 0) return pos - pos % chunk;
+    return window > 0 ? std::max(0, pos - window + 1) : 0;
 }
+
+int KVGroup::first_needed_page(int start_pos) const { return first_key(start_pos) / PAGE; }
 
 std::vector<int> KVGroup::pages_missing(int slot, int start_pos, int new_len) const {
     if (rows_for(new_len) > width * PAGE)
@@ -62,9 +64,9 @@ void KVGroup::reserve(int slot, int start_pos, int new_len) {
 }
 
 void KVGroup::release_behind(int slot, int length) {
-    if (window <= 0) return;
+    if (window <= 0 && chunk <= 0) return;
     int* row = &table[(size_t)slot * width];
-    const int end = std::min(width, std::max(0, length - window + 1) / PAGE);
+    const int end = std::min(width, first_key(length) / PAGE);
     for (int lp = kept_pages(); lp < end; ++lp)
         if (row[lp] >= 0) {
             pages.give(row[lp]);
@@ -100,7 +102,7 @@ Cache::Cache(const std::map<int, CacheRequest>& requests, int64_t max_tokens, in
     // hold more pages than there are, so the table need not be wider than that; with a window it holds few pages
     // at a time but at any logical place.
     const int seq_pages = std::max(1, (max_seq_tokens + PAGE - 1) / PAGE);
-    typedef std::tuple<int, int, int, int, int, int, int> Need;
+    typedef std::tuple<int, int, int, int, int, int, int, int> Need;
     std::vector<std::pair<Need, std::vector<int>>> by_need;          // in order of first appearance
     // a request made of several becomes one request per part, each under a key of its own
     std::map<int, CacheRequest> flat;
@@ -119,8 +121,9 @@ Cache::Cache(const std::map<int, CacheRequest>& requests, int64_t max_tokens, in
         const CacheRequest& r = kv.second;
         if (r.kind == CacheRequest::KV) {
             if (r.every > 1 && r.window > 0) throw CacheError("a cache request with a row per several positions cannot have a window");
+            if (r.chunk > 0 && (r.window > 0 || r.every > 1)) throw CacheError("a cache request with runs of positions cannot have a window, nor a row per several positions");
             const Need need(r.n_kv_heads, r.head_dim, r.window, r.value_dim(), r.keep_first, r.every > 1 ? r.every : 1,
-                            (r.keys_only ? 1 : 0) + (r.store_f32 ? 2 : 0));
+                            (r.keys_only ? 1 : 0) + (r.store_f32 ? 2 : 0), r.chunk);
             auto it = std::find_if(by_need.begin(), by_need.end(), [&](const auto& p) { return p.first == need; });
             if (it == by_need.end()) by_need.emplace_back(need, std::vector<int>{kv.first});
             else it->second.push_back(kv.first);
@@ -141,7 +144,7 @@ Cache::Cache(const std::map<int, CacheRequest>& requests, int64_t max_tokens, in
         const int every = req.every > 1 ? req.every : 1;
         const int group_pages = every > 1 ? (n_pages + every - 1) / every + max_slots : n_pages;
         const int group_seq_pages = every > 1 ? std::max(1, ((max_seq_tokens + every - 1) / every + PAGE - 1) / PAGE) : seq_pages;
-        const int width = req.window > 0 ? group_seq_pages : std::min(group_pages, group_seq_pages);
+        const int width = req.window > 0 || req.chunk > 0 ? group_seq_pages : std::min(group_pages, group_seq_pages);
         groups.emplace_back(new KVGroup(req, p.second, max_slots, group_pages, width, dtype, on_device));
         for (int e : p.second) group_of[e] = (int)groups.size() - 1;
     }
@@ -213,6 +216,7 @@ CacheView Cache::view(int entry, bool write, const std::vector<const int*>& step
         v.table_width = grp.width;
         v.page_size = PAGE;
         v.window = grp.window;
+        v.chunk = grp.chunk;
         v.n_kv_heads = grp.request.n_kv_heads;
         v.head_dim = grp.request.head_dim;
         v.v_head_dim = grp.request.value_dim();

@@ -69,7 +69,10 @@ struct MmaArgs {
     unsigned long long* trace;  // for measurements (may be null): [cta][8] timestamps of a one-token step's CTAs
     // EXTRA only
     FrVec sink;               // [nq]; p null: none
-    const bf16* gate;         // head h's gate of row r at gate[r * q_stride + h]; null: none
+    const bf16* gate;         // head h's gate of row r at gate[r * gate_ld + h]; null: none
+    int gate_ld;
+    int gate_wide;            // 1: a gate per channel instead, channel c of head h at gate[r * gate_ld + h * hd + c]
+    int chunk;                // > 0: a row sees its own run of this many positions only (no window)
     float cap_log2, two_over_cap_log2;   // cap (0: none) and, times the scale, 2 / cap, both in units of log2
 };
 
@@ -78,8 +81,15 @@ template <bool EXTRA>
 __device__ __forceinline__ float row_factor(const MmaArgs& p, float l, float big_log2, int row, int head) {
     if (EXTRA && p.sink.p != nullptr) l += exp2f(fmaf(p.sink.at(head), LOG2E, -big_log2));
     float inv = l > 0.f ? 1.f / l : 0.f;
-    if (EXTRA && p.gate != nullptr) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)row * p.q_stride + head]));
+    if (EXTRA && p.gate != nullptr && !p.gate_wide) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)row * p.gate_ld + head]));
     return inv;
+}
+// the gates of two neighbouring channels of a row's head, where there is a gate per channel
+template <bool EXTRA>
+__device__ __forceinline__ float2 pair_gates(const MmaArgs& p, int row, int head, int hd, int channel) {
+    if (!EXTRA || !p.gate_wide) return make_float2(1.f, 1.f);
+    const uint32_t g = *(const uint32_t*)(p.gate + (size_t)row * p.gate_ld + (size_t)head * hd + channel);
+    return make_float2(1.0f / (1.0f + expf(-__uint_as_float(g << 16))), 1.0f / (1.0f + expf(-__uint_as_float(g & 0xffff0000u))));
 }
 
 __device__ __forceinline__ void mark(const MmaArgs& p, int point) {
@@ -197,7 +207,8 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     // Range of key blocks for this CTA.
     const int t_first = r0 / G, t_last = min((r0 + ROWS_CTA - 1) / G, q_len - 1);
     const int pos_hi = pos0 + t_last;                 // the farthest key any row of the CTA may see
-    const int lo_min = p.window > 0 ? max(0, pos0 + t_first - p.window + 1) : 0;
+    const int chunk = EXTRA ? p.chunk : 0;
+    const int lo_min = fr_first_key(pos0 + t_first, p.window, chunk);
     int kb_begin = lo_min / BLOCK_N, kb_end = pos_hi / BLOCK_N;     // inclusive
     if (p.splits > 1) {
         const int n = kb_end - kb_begin + 1, per = (n + p.splits - 1) / p.splits;
@@ -277,13 +288,13 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
         const int rr = r0 + row_base + (lane >> 2) + 8 * i;
         const bool ok = rr < n_rows;
         pos_r[i] = ok ? pos0 + rr / G : -1;           // -1: every key is masked
-        lo_r[i] = (ok && p.window > 0) ? max(0, pos_r[i] - p.window + 1) : 0;
+        lo_r[i] = ok ? fr_first_key(pos_r[i], p.window, chunk) : 0;
     }
     // Warp-wide bounds that decide whether a block needs the mask at all.
     const int w_first = (r0 + row_base) / G;
     const int w_last = min((r0 + row_base + 15) / G, q_len - 1);
     const int w_pos_min = pos0 + w_first;
-    const int w_lo_max = p.window > 0 ? max(0, pos0 + w_last - p.window + 1) : 0;
+    const int w_lo_max = fr_first_key(pos0 + w_last, p.window, chunk);
 
     float o[DT][4];
 #pragma unroll
@@ -367,7 +378,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
 
         // scale, mask, online softmax
         const int j0 = kb * BLOCK_N + key_base;
-        const bool need_mask = (j0 + KPW - 1 > w_pos_min) || (p.window > 0 && j0 < w_lo_max);
+        const bool need_mask = (j0 + KPW - 1 > w_pos_min) || j0 < w_lo_max;
         float mx[2] = {-INFINITY, -INFINITY};
         const bool capping = EXTRA && p.cap_log2 > 0.f;
 #pragma unroll
@@ -554,8 +565,10 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
                 const int d = d0 + c * V;
                 if (p.splits == 1) {
 #pragma unroll
-                    for (int j = 0; j < V; j += 2)
-                        *reinterpret_cast<uint32_t*>(p.out + item * HD + d + j) = pack_bf16(acc[j] * inv, acc[j + 1] * inv);
+                    for (int j = 0; j < V; j += 2) {
+                        const float2 gt = pair_gates<EXTRA>(p, q_start + t, h, HD, d + j);
+                        *reinterpret_cast<uint32_t*>(p.out + item * HD + d + j) = pack_bf16(acc[j] * inv * gt.x, acc[j + 1] * inv * gt.y);
+                    }
                 } else {
                     float* dst = p.cluster ? r_o + r * HD + d : p.part + (item * p.splits + split) * (HD + 2) + d;
 #pragma unroll
@@ -616,8 +629,9 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
                 const size_t item = (size_t)(q_start + t) * p.nq + h;
                 const float inv = row_factor<EXTRA>(p, l, big, q_start + t, h);
                 uint2 packed;
-                packed.x = pack_bf16(acc.x * inv, acc.y * inv);
-                packed.y = pack_bf16(acc.z * inv, acc.w * inv);
+                const float2 g01 = pair_gates<EXTRA>(p, q_start + t, h, HD, d4 * 4), g23 = pair_gates<EXTRA>(p, q_start + t, h, HD, d4 * 4 + 2);
+                packed.x = pack_bf16(acc.x * inv * g01.x, acc.y * inv * g01.y);
+                packed.y = pack_bf16(acc.z * inv * g23.x, acc.w * inv * g23.y);
                 *reinterpret_cast<uint2*>(p.out + item * HD + d4 * 4) = packed;
             }
             mark(p, 7);
@@ -743,8 +757,9 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
                     }
                     const float inv = s_inv[r2];
                     const int rr2 = r0 + r2, t2 = rr2 / G, h2 = kvh * G + (rr2 - t2 * G);
+                    const float2 gt = pair_gates<EXTRA>(p, q_start + t2, h2, HD, 2 * piece);
                     *reinterpret_cast<uint32_t*>(p.out + ((size_t)(q_start + t2) * p.nq + h2) * HD + 2 * piece) =
-                        pack_bf16(a.x * inv, a.y * inv);
+                        pack_bf16(a.x * inv * gt.x, a.y * inv * gt.y);
                 }
                 mark(p, 7);
             }
@@ -952,15 +967,21 @@ FR_EXPORT int attention_mma(const void* q, int q_stride, void* out, const void* 
 }
 
 // One-token steps with more to their softmax: softcap (0: none), sink [nq] of sink_dtype (null: none), gate: head h's gate of row r
-// at gate[r * q_stride + h], bf16 (null: none).  splits as above, at most 64.
+// at gate[r * gate_ld + h], bf16 (null: none); gate_wide: a gate per channel, channel c of head h at gate[r * gate_ld + h * hd + c].
+// chunk > 0 (window 0): a row sees its own run of `chunk` positions only.  splits as above, at most 64.
 FR_EXPORT int attention_mma_extra(const void* q, int q_stride, void* out, const void* k_pool, const void* v_pool, int pool_pages,
                                   const int* block_table, int table_width, int page, const int* seq_start,
                                   const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int rows, int nq, int nkv, int hd,
-                                  int window, float scale, float softcap, const void* sink, int sink_dtype, const void* gate, int splits,
-                                  float* scratch, int* counters, int n_counters, int* status, cudaStream_t stream) {
+                                  int window, float scale, float softcap, const void* sink, int sink_dtype, const void* gate, int gate_ld,
+                                  int gate_wide, int chunk, int splits, float* scratch, int* counters, int n_counters, int* status, cudaStream_t stream) {
     MmaArgs e{};
     e.sink = FrVec{sink, sink_dtype};
     e.gate = (const bf16*)gate;
+    e.gate_ld = gate_ld;
+    e.gate_wide = gate != nullptr && gate_wide;
+    e.chunk = chunk;
+    if (chunk < 0 || (chunk > 0 && window > 0)) FR_REFUSE("attention_mma: chunks of %d positions beside a window of %d", chunk, window);
+    if (e.gate_wide && (gate_ld % 2 || ((uintptr_t)gate & 3))) FR_REFUSE("attention_mma: gates per channel lie in whole pairs");
     e.cap_log2 = softcap * LOG2E;
     e.two_over_cap_log2 = softcap > 0.f ? 2.0f * scale * LOG2E / softcap : 0.f;
     return attention_mma_run(q, q_stride, out, k_pool, v_pool, pool_pages, block_table, table_width, page, seq_start, seq_qlen, seq_pos0,

@@ -8,7 +8,8 @@
 // b P .. b P + P - 1) if b P + P - 1 <= i - window: the first floor(max(0, i - window + 1) / P) blocks.  Tokens and blocks
 // share one softmax; with a sink s_h the denominator also holds exp(s_h).  Head h's scores are (q . k) * scale * m(i) with
 // m(i) = 1 + coef * ln(floor((i + 1) / every) + 1), the multiplier applied to the 32-bit score, not to the stored query; with a cap
-// c a score s becomes c tanh(s / c).  Head h's result is multiplied by sigmoid(gate_h) where the rows carry gates.
+// c a score s becomes c tanh(s / c).  Head h's result is multiplied by sigmoid(gate_h), or element by element by the sigmoid of a
+// gate per channel, where the rows carry gates.  With a chunk size C row i sees token j <= i if floor(i / C) = floor(j / C) instead.
 //
 //   prepare   per row: q and k heads are RMS-normed with a weight shared by the heads (optional), the first `rot` numbers
 //             of each head turn by position (pairs (i, i + rot / 2), angle fp32(pos) * freq[i], cosine and sine times a
@@ -329,7 +330,9 @@ struct RowArgs {
     const int* row_pos;
     FrVec sink;              // [heads]; p null: none
     float* part;             // [rows][heads][splits][vdim + 2]
-    const void* gate;        // head h's gate of row r at gate[r * q_stride + h]; null: none
+    const void* gate;        // head h's gate of row r at gate[r * gate_ld + h]; null: none
+    int gate_ld, gate_wide;  // gate_wide: a gate per channel instead, channel c of head h at gate[r * gate_ld + h * vdim + c]
+    int chunk;               // > 0: row i sees the tokens of its own run of this many positions only (no window)
     int table_width, pool_table_width, rows, heads, kv_heads, dim, vdim, q_stride, q_off, window, pool, splits, temp_every;
     float scale, temp_coef, softcap;
 };
@@ -404,7 +407,7 @@ __global__ void __launch_bounds__(128) rows_kernel(RowArgs p) {
     float m = -INFINITY, l = 0.f;
     if (seq >= 0) {
         const int pos = p.row_pos[row], kvh = h / (p.heads / p.kv_heads);
-        const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+        const int lo = fr_first_key(pos, p.window, p.chunk);
         const int n_blocks = blocks_in_sight(pos, p.window, p.pool);
         const int n = n_blocks + pos - lo + 1;
         const int chunk = (n + p.splits - 1) / p.splits;
@@ -468,12 +471,13 @@ __global__ void __launch_bounds__(128) rows_merge_kernel(RowArgs p) {
         }
     }
     float inv = l > 0.f ? 1.0f / l : 0.f;
-    if (p.gate != nullptr) inv /= 1.0f + expf(-fr_load((const T*)p.gate + (size_t)(item / p.heads) * p.q_stride + h));
+    const T* gates = (const T*)p.gate + (size_t)(item / p.heads) * p.gate_ld + (p.gate_wide ? (size_t)h * p.vdim : (size_t)h);
+    if (p.gate != nullptr && !p.gate_wide) inv /= 1.0f + expf(-fr_load(gates));
     T* o_row = (T*)p.out + (size_t)item * p.vdim;
 #pragma unroll
     for (int i = 0; i < MAX_PER_LANE; ++i) {
         const int d = lane + 32 * i;
-        if (d < p.vdim) fr_store(o_row + d, acc[i] * inv);
+        if (d < p.vdim) fr_store(o_row + d, p.gate_wide ? acc[i] * inv / (1.0f + expf(-fr_load(gates + d))) : acc[i] * inv);
     }
 }
 
@@ -493,7 +497,8 @@ struct PromptArgs {
     const int* seq_qlen;
     const int* seq_pos0;
     FrVec sink;
-    const bf16* gate;        // head h's gate of row r at gate[r * q_stride + h]; null: none
+    const bf16* gate;        // head h's gate of row r at gate[r * gate_ld + h]; null: none
+    int gate_ld, gate_wide, chunk;      // as in RowArgs
     int table_width, pool_table_width, q_stride, q_off, heads, kv_heads, dim, vdim, window, pool, temp_every;
     float scale, temp_coef, softcap;
 };
@@ -573,7 +578,8 @@ __global__ void __launch_bounds__(128, 3) prompt_kernel(PromptArgs p) {
                            p.scale * query_multiplier(my_pos[1], p.temp_coef, p.temp_every)};
     const int my_blocks[2] = {blocks_in_sight(my_pos[0], p.window, p.pool), blocks_in_sight(my_pos[1], p.window, p.pool)};
 
-    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;             // earliest token that the first row sees
+    const int lo = fr_first_key(pos0, p.window, p.chunk);                      // earliest token that the first row sees
+    const int my_lo[2] = {fr_first_key(my_pos[0], p.window, p.chunk), fr_first_key(my_pos[1], p.window, p.chunk)};
     const int pooled_rows = blocks_in_sight(last_pos, p.window, p.pool);       // pooled blocks that the last row sees
     const int pooled_tiles = (pooled_rows + BN - 1) / BN;
     const int first_block = lo / BN, last_block = last_pos / BN;
@@ -626,7 +632,7 @@ __global__ void __launch_bounds__(128, 3) prompt_kernel(PromptArgs p) {
             for (int e = 0; e < 4; ++e) {
                 const int j = b * BN + nt * 8 + 2 * t + (e & 1), half = e >> 1;
                 const int pos = my_pos[half];
-                const bool seen = pos <= last_pos && (pooled ? j < my_blocks[half] : (j <= pos && (p.window <= 0 || pos - j < p.window)));
+                const bool seen = pos <= last_pos && (pooled ? j < my_blocks[half] : (j <= pos && j >= my_lo[half]));
                 float v = s[nt][e] * mult[half];
                 if (capping) v = fr_capped(v, p.softcap, two_over_cap);
                 s[nt][e] = seen ? v : -INFINITY;
@@ -694,12 +700,17 @@ __global__ void __launch_bounds__(128, 3) prompt_kernel(PromptArgs p) {
             l = l * f + expf(sink - big);
         }
         float inv = l > 0.f ? f / l : 0.f;
-        if (p.gate != nullptr) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)(row0 + r) * p.q_stride + h]));
+        const bf16* gates = p.gate + (size_t)(row0 + r) * p.gate_ld + (p.gate_wide ? (size_t)h * p.vdim : (size_t)h);
+        if (p.gate != nullptr && !p.gate_wide) inv /= 1.0f + expf(-__bfloat162float(*gates));
         bf16* dst = p.out + (size_t)(row0 + r) * p.heads * p.vdim + (size_t)h * p.vdim;
 #pragma unroll
         for (int nt = 0; nt < DV / 8; ++nt) {
             const int c = nt * 8 + 2 * t;
-            const float x = o[nt][2 * half] * inv, y = o[nt][2 * half + 1] * inv;
+            float x = o[nt][2 * half] * inv, y = o[nt][2 * half + 1] * inv;
+            if (p.gate_wide) {
+                if (c < p.vdim) x /= 1.0f + expf(-__bfloat162float(gates[c]));
+                if (c + 1 < p.vdim) y /= 1.0f + expf(-__bfloat162float(gates[c + 1]));
+            }
             if (c + 1 < p.vdim && (((uintptr_t)(dst + c)) & 3) == 0) *(uint32_t*)(dst + c) = pack2(x, y);
             else {
                 if (c < p.vdim) dst[c] = __float2bfloat16_rn(x);
@@ -803,13 +814,14 @@ FR_EXPORT long long attention_pooled_scratch_floats(int rows, int heads, int vdi
 
 // q [rows][q_stride] and out [rows][heads * vdim] of `dtype`, like the token pools; the pooled pools are fp32 sums (null with
 // pool 0).  sink [heads] of sink_dtype (null: none).  temp_every 0: no query multiplier; softcap 0: none.  gate: head h's gate of
-// row r at gate[r * q_stride + h], in the rows' dtype (null: none).
+// row r at gate[r * gate_ld + h], in the rows' dtype (null: none), or with gate_wide a gate per channel, channel c of head h at
+// gate[r * gate_ld + h * vdim + c].  chunk > 0 (window and pool 0): a row sees its own run of `chunk` positions only.
 FR_EXPORT int attention_pooled_rows(const void* q, int q_stride, int q_off, void* out, const void* k_pool, const void* v_pool,
                                     const float* pk_pool, const float* pv_pool, const int* block_table, int table_width,
                                     const int* pool_table, int pool_table_width, int page, const int* row_seq, const int* row_pos, int rows,
                                     int heads, int kv_heads, int dim, int vdim, int window, int pool, float scale, float temp_coef,
-                                    int temp_every, float softcap, const void* sink, int sink_dtype, const void* gate, int splits,
-                                    float* scratch, int dtype, cudaStream_t stream) {
+                                    int temp_every, float softcap, const void* sink, int sink_dtype, const void* gate, int gate_ld, int gate_wide,
+                                    int chunk, int splits, float* scratch, int dtype, cudaStream_t stream) {
     if (rows <= 0) return FR_OK;
     const int rc = check_shape(heads, kv_heads, dim, vdim, window, pool, page);
     if (rc != FR_OK) return rc;
@@ -820,7 +832,8 @@ FR_EXPORT int attention_pooled_rows(const void* q, int q_stride, int q_off, void
     p.pool_table = pool_table; p.row_seq = row_seq; p.row_pos = row_pos; p.sink = FrVec{sink, sink_dtype}; p.part = scratch;
     p.table_width = table_width; p.pool_table_width = pool_table_width; p.rows = rows; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim;
     p.vdim = vdim; p.q_stride = q_stride; p.q_off = q_off; p.window = window; p.pool = pool; p.splits = splits; p.temp_every = temp_every;
-    p.scale = scale; p.temp_coef = temp_coef; p.softcap = softcap; p.gate = gate;
+    p.scale = scale; p.temp_coef = temp_coef; p.softcap = softcap; p.gate = gate; p.gate_ld = gate_ld; p.gate_wide = gate != nullptr && gate_wide; p.chunk = chunk;
+    if (chunk < 0 || (chunk > 0 && window > 0)) FR_REFUSE("attention_pooled: chunks of %d positions beside a window of %d", chunk, window);
     const int items = rows * heads;
     const dim3 grid((items + 3) / 4, splits), mgrid((items + 3) / 4);
     if (dtype == FR_F32) {
@@ -844,7 +857,7 @@ FR_EXPORT int attention_pooled_prompt(const void* q, int q_stride, int q_off, vo
                                       const int* pool_table, int pool_table_width, int page, const int* seq_start, const int* seq_qlen,
                                       const int* seq_pos0, int n_seqs, int max_q_len, int heads, int kv_heads, int dim, int vdim, int window,
                                       int pool, float scale, float temp_coef, int temp_every, float softcap, const void* sink, int sink_dtype,
-                                      const void* gate, cudaStream_t stream) {
+                                      const void* gate, int gate_ld, int gate_wide, int chunk, cudaStream_t stream) {
     if (n_seqs <= 0 || max_q_len <= 0) return FR_OK;
     const int rc = check_shape(heads, kv_heads, dim, vdim, window, pool, page);
     if (rc != FR_OK) return rc;
@@ -856,7 +869,9 @@ FR_EXPORT int attention_pooled_prompt(const void* q, int q_stride, int q_off, vo
     p.block_table = block_table; p.pool_table = pool_table; p.seq_start = seq_start; p.seq_qlen = seq_qlen; p.seq_pos0 = seq_pos0;
     p.sink = FrVec{sink, sink_dtype}; p.table_width = table_width; p.pool_table_width = pool_table_width; p.q_stride = q_stride; p.q_off = q_off;
     p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.pool = pool; p.temp_every = temp_every;
-    p.scale = scale; p.temp_coef = temp_coef; p.softcap = softcap; p.gate = (const bf16*)gate;
+    p.scale = scale; p.temp_coef = temp_coef; p.softcap = softcap; p.gate = (const bf16*)gate; p.gate_ld = gate_ld;
+    p.gate_wide = gate != nullptr && gate_wide; p.chunk = chunk;
+    if (chunk < 0 || (chunk > 0 && window > 0)) FR_REFUSE("attention_pooled: chunks of %d positions beside a window of %d", chunk, window);
     if (dim <= 32) return prompt_by_value_size<32>(p, n_seqs, max_q_len, stream);
     if (dim <= 64) return prompt_by_value_size<64>(p, n_seqs, max_q_len, stream);
     return prompt_by_value_size<128>(p, n_seqs, max_q_len, stream);

@@ -77,6 +77,8 @@ struct TcArgs {
     FrVec sink;               // [nq]; p null: none
     const bf16* gate;         // head h's gate of row r at gate[r * gate_ld + h]; null: none
     int gate_ld;
+    int gate_wide;            // 1: a gate per channel instead, channel c of head h at gate[r * gate_ld + h * vd + c]
+    int chunk;                // > 0: a row sees its own run of this many positions only (no window)
     float cap_log2, two_over_cap_log2;   // cap (0: none) and, times the scale, 2 / cap, both in units of log2
     unsigned long long* trace;   // for measurements (may be null): [cta][8] sums of time (ns) that row 0's thread spent
                                  // waiting for S, reading it, writing P, rescaling O, waiting for the last product;
@@ -153,9 +155,12 @@ __device__ __forceinline__ void scale_and_cap(const TcArgs& p, uint32_t (&raw)[N
 __device__ __forceinline__ float row_factor(const TcArgs& p, float l, float m, int row, int head) {
     if (p.sink.p != nullptr) l += exp2f(fmaf(p.sink.at(head), LOG2E, -m));
     float inv = l > 0.f ? 1.f / l : 0.f;
-    if (p.gate != nullptr) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)row * p.gate_ld + head]));
+    if (p.gate != nullptr && !p.gate_wide) inv /= 1.0f + expf(-__bfloat162float(p.gate[(size_t)row * p.gate_ld + head]));
     return inv;
 }
+
+// the sigmoid of a gate that is about to be rounded to bf16
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + exp2_fast(-LOG2E * z)); }
 
 __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -229,7 +234,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     if (p.seq_live != nullptr && p.seq_live[q_start] < 0) return;     // an ended sequence's rows are not written
     const int t_end = min(t0 + T, q_len);             // tokens t0 .. t_end-1
     const int pos_hi = pos0 + t_end - 1;              // the farthest key any row of the CTA may see
-    const int lo_min = p.window > 0 ? max(0, pos0 + t0 - p.window + 1) : 0;
+    const int chunk = EXTRA ? p.chunk : 0;
+    const int lo_min = fr_first_key(pos0 + t0, p.window, chunk);      // the first key of the first row, and of the last
+    const int lo_max = fr_first_key(pos_hi, p.window, chunk);
     const int kb_begin = lo_min / KEYS, kb_end = pos_hi / KEYS;       // inclusive
     const int n_blocks = kb_end - kb_begin + 1;
     const int slices = (p.hd + 63) / 64, vslices = (p.vd + 63) / 64;
@@ -366,7 +373,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int t = r / G, g = r - t * G;
         const bool valid = r < T * G && t0 + t < q_len;
         const int pos_r = valid ? pos0 + t0 + t : -1;      // -1: every key is masked
-        const int lo_r = (valid && p.window > 0) ? max(0, pos_r - p.window + 1) : 0;
+        const int lo_r = valid ? fr_first_key(pos_r, p.window, chunk) : 0;
         const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
         float m_run = -INFINITY, l_run = 0.f;              // the maximum that P is taken against, and the sum of P
         bool ok = true;
@@ -395,8 +402,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             // tensor memory and is never written.  With them in the condition the warp of the tile's last rows, two of
             // which are such rows when 7 heads share a kv head, took the masked form in every block, 2.5 times as long
             // as the others.)
-            const bool need_mask = __any_sync(0xffffffffu, j0 + KEYS - 1 > pos0 + t0 ||
-                                                               (p.window > 0 && j0 < pos_hi - p.window + 1));
+            const bool need_mask = __any_sync(0xffffffffu, j0 + KEYS - 1 > pos0 + t0 || j0 < lo_max);
             uint32_t raw[KEYS];
             {
                 uint32_t (&lo32)[32] = *reinterpret_cast<uint32_t (*)[32]>(&raw[0]);
@@ -504,6 +510,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         if (ok) {
             const float inv = !valid ? 0.f : EXTRA ? row_factor(p, l_run, m_run, q_start + t0 + t, kvh * G + g) : l_run > 0.f ? 1.f / l_run : 0.f;
             bf16* dst = p.out + ((size_t)(q_start + t0 + t) * p.nq + (size_t)kvh * G + g) * p.vd;
+            const bf16* gates = EXTRA && p.gate_wide ? p.gate + (size_t)(q_start + t0 + t) * p.gate_ld + (size_t)(kvh * G + g) * p.vd : nullptr;
 #pragma unroll 1
             for (int c = 0; c < 4; ++c) {
                 if (c * 32 < p.vd) {                                   // uniform: the load is warp-wide
@@ -517,6 +524,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                                 float x[8];
 #pragma unroll
                                 for (int j = 0; j < 8; ++j) x[j] = __uint_as_float(o32[q * 8 + j]) * inv;
+                                if (EXTRA && gates != nullptr) {
+                                    const uint4 gr = *(const uint4*)(gates + c * 32 + q * 8);
+                                    const uint32_t gw[4] = {gr.x, gr.y, gr.z, gr.w};
+#pragma unroll
+                                    for (int j = 0; j < 4; ++j) {
+                                        x[2 * j] *= sigmoid_fast(__uint_as_float(gw[j] << 16));
+                                        x[2 * j + 1] *= sigmoid_fast(__uint_as_float(gw[j] & 0xffff0000u));
+                                    }
+                                }
                                 *(uint4*)(dst + c * 32 + q * 8) =
                                     make_uint4(pack2(x[0], x[1]), pack2(x[2], x[3]), pack2(x[4], x[5]), pack2(x[6], x[7]));
                             }
@@ -1042,12 +1058,14 @@ FR_EXPORT int attention_tc(const void* q, int q_stride, int total_rows, void* ou
 }
 
 // The form with more to its softmax: values of vd numbers (out [rows][nq * vd], value pool [pool_pages][64][nkv][vd]), softcap (0:
-// none), sink [nq] of sink_dtype (null: none), gate: head h's gate of row r at gate[r * gate_ld + h], bf16 (null: none).
+// none), sink [nq] of sink_dtype (null: none), gate: head h's gate of row r at gate[r * gate_ld + h], bf16 (null: none); gate_wide: a
+// gate per channel, channel c of head h at gate[r * gate_ld + h * vd + c].  chunk > 0 (window 0): a row sees its own run of `chunk`
+// positions only.
 FR_EXPORT int attention_tc_extra(const void* q, int q_stride, int total_rows, void* out, const void* k_pool, const void* v_pool,
                                  int pool_pages, const int* block_table, int table_width, const int* seq_start,
                                  const int* seq_qlen, const int* seq_pos0, const int* seq_live, int n_seqs, int max_q_len,
                                  int nq, int nkv, int hd, int vd, int window, float scale, float softcap, const void* sink, int sink_dtype,
-                                 const void* gate, int gate_ld, int* status, cudaStream_t stream) {
+                                 const void* gate, int gate_ld, int gate_wide, int chunk, int* status, cudaStream_t stream) {
     if (n_seqs <= 0 || total_rows <= 0 || max_q_len <= 0) return FR_OK;
     TcArgs p;
     CUtensorMap mq, mk, mv;
@@ -1057,6 +1075,10 @@ FR_EXPORT int attention_tc_extra(const void* q, int q_stride, int total_rows, vo
     p.sink = FrVec{sink, sink_dtype};
     p.gate = (const bf16*)gate;
     p.gate_ld = gate_ld;
+    p.gate_wide = gate != nullptr && gate_wide;
+    p.chunk = chunk;
+    if (chunk < 0 || (chunk > 0 && window > 0)) FR_REFUSE("attention_tc: chunks of %d positions beside a window of %d", chunk, window);
+    if (p.gate_wide && ((gate_ld | vd) % 8 || ((uintptr_t)gate & 15))) FR_REFUSE("attention_tc: gates per channel lie in whole 16-byte pieces");
     p.cap_log2 = softcap * LOG2E;
     p.two_over_cap_log2 = softcap > 0.f ? 2.0f * scale * LOG2E / softcap : 0.f;
     return launch<true>(mq, mk, mv, p, max_q_len, stream);

@@ -108,6 +108,13 @@ __device__ __forceinline__ float fr_capped(float raw, float cap, float two_over_
     return fmaf(-2.0f * cap, r, cap);
 }
 
+// The first position that a query at `pos` sees: the start of its own run of `chunk` positions (counted from position 0 of the
+// sequence), or the far end of its window, or 0 where neither is set.  It never falls as `pos` grows.
+__host__ __device__ __forceinline__ int fr_first_key(int pos, int window, int chunk) {
+    if (chunk > 0) return pos - pos % chunk;
+    return window > 0 && pos >= window ? pos - window + 1 : 0;
+}
+
 // The rotation of one pair of a rotary encoding, the same instructions wherever it is applied.
 __device__ __forceinline__ void fr_rotate(float a, float b, float c, float s, float& ra, float& rb) {
     ra = __fmaf_rn(-b, s, __fmul_rn(a, c));

@@ -18,10 +18,9 @@
 #include <math.h>
 
 #include "common.cuh"
+#include "mma_sync.cuh"
 
 FR_EXPORT const char* linear_decay_last_error() { return fr_error_text; }
-
-typedef __nv_bfloat16 bf16;
 
 namespace {
 
@@ -109,42 +108,9 @@ __global__ void __launch_bounds__(256) scan_kernel(DecayArgs p) {
 }
 
 // ------------------------------------------------------------------ chunks on the tensor cores
-__device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const bf16* p) {
-    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const bf16* p) {
-    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
-}
-__device__ __forceinline__ uint32_t pack2(float x, float y) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
-    return *(const uint32_t*)&v;
-}
-// head and remainder of two fp32 numbers as packed bf16 pairs
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-    const bf16 hx = __float2bfloat16_rn(x), hy = __float2bfloat16_rn(y);
-    const __nv_bfloat162 h = __halves2bfloat162(hx, hy);
-    hi = *(const uint32_t*)&h;
-    lo = pack2(x - __bfloat162float(hx), y - __bfloat162float(hy));
-}
 constexpr int THR = 256;             // threads of a chunk's block
 
-// channels c .. c + 7 of a row of n channels (zero beyond) as stored
-__device__ __forceinline__ uint4 raw8(const bf16* src, int c, int n) {
-    if (c + 8 <= n && (((uintptr_t)(src + c)) & 15) == 0) return *(const uint4*)(src + c);
-    uint4 v = make_uint4(0, 0, 0, 0);
-    bf16* e = (bf16*)&v;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) e[i] = c + i < n ? src[c + i] : __float2bfloat16_rn(0.f);
-    return v;
-}
-// their silu, fp32 values that bf16 holds exactly
+// the silu of eight channels, fp32 values that bf16 holds exactly
 __device__ __forceinline__ void silu8(const uint4& r, float (&v)[8]) {
     const uint32_t w[4] = {r.x, r.y, r.z, r.w};
 #pragma unroll

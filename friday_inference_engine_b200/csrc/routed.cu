@@ -6,6 +6,7 @@
 //   scale_by_route   act [rows][experts * inner] *= dense[row][column / inner]: after it, one product over all
 //                    experts' down matrices side by side sums exactly the chosen experts
 //   route_biased     softmax scores over experts and identity experts (which return their input), a bias for the choice only
+//   route_table      no router: a table gives each token id its experts, all with the weight 1 / top
 //   shared_and_self  the row's gate times the shared expert's result, plus what its identity experts weigh times the row
 //   gate_up          for every (row, choice): act = silu(Wg_e h) * (Wu_e h) (or the clipped unit), expert e's rows read where they lie
 //   down_combine     out[row] = residual[row] + sum over choices of weight * (Wd_e act)
@@ -95,6 +96,28 @@ route_kernel(const float* __restrict__ logits, int ld, int rows, int experts, in
         weights[(size_t)row * top + lane] = w;
         if (dense != nullptr && my_id >= 0) dense[(size_t)row * experts + my_id] = w;
     }
+}
+
+// a warp per row
+__global__ void __launch_bounds__(128)
+route_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table, int vocab, int rows, int experts, int top, int* __restrict__ ids,
+                   float* __restrict__ weights, float* __restrict__ dense) {
+    fr_pdl_wait();
+    fr_pdl_launch();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int row = blockIdx.x * 4 + warp;
+    if (row >= rows) return;
+    const int token = tokens[row];
+    if (dense != nullptr)
+        for (int e = lane; e < experts; e += 32) dense[(size_t)row * experts + e] = 0.f;
+    __syncwarp();
+    if (lane >= top) return;
+    int id = token >= 0 && token < vocab ? table[(size_t)token * top + lane] : -1;
+    if (id < 0 || id >= experts) id = -1;
+    const float w = 1.0f / (float)top;
+    ids[(size_t)row * top + lane] = id;
+    weights[(size_t)row * top + lane] = w;
+    if (dense != nullptr && id >= 0) dense[(size_t)row * experts + id] = w;
 }
 
 // one row per blockIdx.y; eight consecutive channels per thread where rows allow 16-byte pieces
@@ -808,6 +831,17 @@ FR_EXPORT int routed_route_biased(const float* logits, int ld, int rows, int exp
 }
 
 // gate: the logits' column that holds the rows' gates, gate_ld apart from row to row
+// tokens [rows]: token ids below `vocab`; table [vocab][top]: the experts of every id (an entry that is no expert counts as none);
+// ids, weights [rows][top]; dense (may be null) [rows][experts]
+FR_EXPORT int routed_route_table(const int* tokens, const int* table, int vocab, int rows, int experts, int top, int* ids, float* weights, float* dense,
+                                 cudaStream_t stream) {
+    if (rows <= 0) return FR_OK;
+    if (experts < 1 || top < 1 || top > experts || top > 32 || vocab < 1) FR_REFUSE("route: top %d of %d experts (at most 32), %d token ids", top, experts, vocab);
+    FR_CUDA(fr_launch(route_table_kernel, dim3((rows + 3) / 4), dim3(128), 0, stream, tokens, table, vocab, rows, experts, top, ids, weights, dense));
+    FR_CHECK_LAUNCH("route_table");
+    return FR_OK;
+}
+
 FR_EXPORT int routed_shared_and_self(const float* residual, const float* shared, const float* gate, int gate_ld, const float* self, const void* h,
                                      float* out, int rows, int width, int dtype, cudaStream_t stream) {
     if (rows <= 0 || width <= 0) return FR_OK;

@@ -86,6 +86,7 @@ Json request_json(const CacheRequest& r) {
         j.set("window", Json(r.window));
         j.set("v_head_dim", Json(r.value_dim()));
         j.set("keep_first", Json(r.keep_first));
+        if (r.chunk > 0) j.set("chunk", Json(r.chunk));
         if (r.every > 1) j.set("every", Json(r.every));              // what only some mixers ask for is named only then
         if (r.keys_only) j.set("keys_only", Json(true));
         if (r.store_f32) j.set("store_f32", Json(true));
@@ -106,6 +107,7 @@ CacheRequest request_from(const Json& j) {
         CacheRequest r = CacheRequest::kv((int)j.get_int("n_kv_heads", 0), (int)j.get_int("head_dim", 0), (int)j.get_int("window", 0),
                                           (int)j.get_int("v_head_dim", 0), (int)j.get_int("keep_first", 0));
         r.every = (int)j.get_int("every", 1);
+        r.chunk = (int)j.get_int("chunk", 0);
         r.keys_only = j.get_bool("keys_only", false);
         r.store_f32 = j.get_bool("store_f32", false);
         return r;

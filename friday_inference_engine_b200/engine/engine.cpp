@@ -169,6 +169,7 @@ size_t Stepper::step(const StepBatch& b, float* out, bool out_on_device) {
         ctx.n_seqs = (int)nseq;
         ctx.slots = slots;
         ctx.q_lens = q_lens;
+        ctx.host_tokens.assign(host + offs[0], host + offs[0] + rows);
         ctx.max_q_len = *std::max_element(q_lens.begin(), q_lens.end());
         for (size_t k = 0; k < nseq; ++k) ctx.kv_lens.push_back(start[k] + q_lens[k]);
         ctx.max_kv_len = *std::max_element(ctx.kv_lens.begin(), ctx.kv_lens.end());

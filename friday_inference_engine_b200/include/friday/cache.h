@@ -19,6 +19,8 @@
 // own.  Every state request gets a tensor [slots, *shape]
 // that is zeroed when a slot is taken.  A request with `every` = P > 1 keeps one row for every P positions (a mixer's
 // pooled blocks): its group counts a sequence of n tokens as ceil(n / P) rows, has fewer pages accordingly and no window;
+// A group whose positions see their own run of `chunk` positions only gives a page back as soon as the sequence's next position
+// begins a run behind it.
 // `store_f32` keeps its rows in 32-bit, `keys_only` leaves the value pool out.  Lengths, not contents, decide what is valid:
 // slots and pages are used again without being cleared.
 //
@@ -67,7 +69,7 @@ public:
     int rows_for(int tokens) const { return (tokens + every() - 1) / every(); }       // rows that `tokens` positions take
     CacheRequest request;
     std::vector<int> entries;        // cache entry ids, in pool order
-    int window, n_pages, width;
+    int window, chunk, n_pages, width;
     DType dtype;
     FreeList pages;
     std::vector<int> table;          // [slots][width]
@@ -77,6 +79,7 @@ public:
     size_t entry_bytes() const { return (size_t)n_pages * PAGE * request.n_kv_heads * request.head_dim * dtype_size(dtype); }
     size_t value_entry_bytes() const { return request.keys_only ? 0 : (size_t)n_pages * PAGE * request.n_kv_heads * request.value_dim() * dtype_size(dtype); }
     int kept_pages() const { return window > 0 ? (request.keep_first + PAGE - 1) / PAGE : 0; }    // never given back behind the window
+    int first_key(int pos) const;                                   // the earliest position that a query at pos sees
     int first_needed_page(int start_pos) const;                     // logical page of the earliest key a query at start_pos or later sees
     std::vector<int> pages_missing(int slot, int start_pos, int new_len) const;
     void reserve(int slot, int start_pos, int new_len);

@@ -246,12 +246,44 @@ public:
         // columns of the stacked projection; v_off < 0: the values are the keys; k_off < 0: queries only (another layer's keys and values)
         int64_t q_off = 0, k_off = 0, v_off = -1;
         int64_t gate_off = -1;          // >= 0: head h's result is multiplied by sigmoid of column gate_off + h
+        bool gate_wide = false;         // a gate per channel instead: channel c of head h by sigmoid of column gate_off + h * vdim + c
+        const Tensor* gate_rows = nullptr;      // where the gate columns are, if not in the rows that hold the queries
+        int chunk = 0;                  // > 0: row i sees token j <= i if floor(i / chunk) = floor(j / chunk) (no window, no pooled blocks)
     };
     // q (normed, rotated) goes back into proj; k (normed, rotated) and v go to the cache rows of the step's tokens; with
     // pooled blocks the blocks' sums (`pooled`: a view of 32-bit rows, one per `pool` positions) take the step's tokens
     void pooled_store(Tensor& proj, const PooledSpec& spec, const CacheView& tokens, const CacheView* pooled, const StepContext& ctx);
     // -> [rows, heads * vdim] in proj's dtype
     Tensor pooled_attention(const Tensor& proj, const PooledSpec& spec, const CacheView& tokens, const CacheView* pooled, const StepContext& ctx);
+
+    // ---- a short causal convolution per channel over time, and what follows it at once (csrc/short_conv.cu)
+    // The state (`view`, fp32) keeps the last taps - 1 inputs [taps - 1][channels] from hist_off on; taps [channels, n].
+    struct ConvSpec {
+        int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+        int64_t off = 0, hist_off = 0;  // first channel's column of the rows
+        const float* freq = nullptr;    // device [rot / 2]: pairs (2i, 2i + 1) of q and k turn by pos * freq[i] after the convolution
+        int rot = 0;
+        bool unit_norm = false;         // then every q and k head is divided by sqrt(its mean square + eps)
+        float eps = 1e-5f;
+    };
+    // Columns off, off + 1, ... of proj are query heads, key heads and value heads: returns the queries [rows, heads * dim]; keys and
+    // values go to the cache rows of the step's tokens.
+    Tensor conv_heads(const Tensor& proj, const Tensor& taps, const ConvSpec& spec, const CacheView& tokens, const CacheView& state, const StepContext& ctx);
+    // silu(conv + bias) of `channels` columns from `off` on -> [rows, channels] of `dtype`
+    Tensor conv_silu_rows(const Tensor& proj, int64_t off, int64_t channels, const Tensor& taps, const Tensor* bias, const CacheView& state, int64_t hist_off,
+                          DType dtype, const StepContext& ctx);
+
+    // ---- state space duality (csrc/ssd.cu): S <- exp(-exp(a_log) dt) S + dt B x^T per head, y = S^T C + skip x, dt = softplus(raw + dt_bias)
+    struct SsdSpec {
+        int heads = 0, groups = 0, state = 0, vdim = 0;     // S [state][vdim]; head h reads B and C of group h / (heads / groups)
+        int64_t x_off = 0, b_off = 0, c_off = 0;            // columns of xbc: x [heads * vdim], B and C [groups * state]
+        int64_t s_off = 0;                                  // floats before the heads' matrices in a sequence's state
+    };
+    // dt: 32-bit rows whose first `heads` columns are the raw step sizes -> [rows, heads * vdim] fp32
+    Tensor ssd_scan(const Tensor& xbc, const Tensor& dt, const Tensor& dt_bias, const Tensor& a_log, const Tensor& skip, const SsdSpec& spec,
+                    const CacheView& state, const StepContext& ctx);
+    // y [rows, n] fp32 times silu(z); each of `parts` equal runs of a row divided by sqrt(its mean square + eps); times weight, in `dtype`
+    Tensor gate_group_norm(const Tensor& y, const Tensor& z, const Tensor& weight, int parts, float eps, DType dtype);
 
     // ---- attention over a cached latent (csrc/attention_latent.cu)
     struct LatentSpec {
@@ -292,6 +324,8 @@ public:
     // the chosen scores divided by their sum + 1e-20.  A chosen identity expert (the last `identity` of them) has id -1 and adds its
     // weight to `self`.
     Routing route_biased(const Tensor& logits, int experts, int identity, int top, const Tensor* bias, bool with_dense);
+    // No router: table [vocab, top] int32 gives each token id its experts, every one with the weight 1 / top
+    Routing route_table(const int* tokens, int64_t rows, const Tensor& table, int experts, bool with_dense);
     // residual (null: none) + sigmoid(gate column of the logits) * shared (null: none) + self * h, 32-bit rows
     Tensor shared_and_self(const Tensor* residual, const Tensor* shared, const Tensor* logits, int64_t gate_col, const Tensor* self, const Tensor& h);
     void scale_by_route(Tensor& act, const Tensor& dense, int experts, int inner);
@@ -299,11 +333,11 @@ public:
                           float slope = 1.f);
     Tensor expert_down_combine(const Tensor& act, const Routing& r, const Tensor& w_down, const Tensor& residual, int top, int inner);
     // Many rows: the rows are gathered expert by expert and every expert with rows runs its two products on the tensor
-    // cores over its own rows only.  The host reads the experts' row counts (one small copy and a wait per call), so this
-    // is for prompts, never inside a captured step.  w_gate_up [experts * 2 * inner, width] (gate and up row by row in
+    // cores over its own rows only.  The host reads the experts' row counts (one small copy and a wait per call) unless it knows
+    // them already (`counts`: a number of choices per expert), so this is for prompts, never inside a captured step.  w_gate_up [experts * 2 * inner, width] (gate and up row by row in
     // turn), w_down [width, experts * inner].
     Tensor experts_grouped(const Tensor& h, const Routing& r, const Tensor& w_gate_up, const Tensor& w_down, const Tensor& residual,
-                           int top, int inner, int act = 1, float limit = 0.f, float slope = 1.f);
+                           int top, int inner, int act = 1, float limit = 0.f, float slope = 1.f, const std::vector<int>* counts = nullptr);
 
     // ---- matrix products: x [rows, k] @ weight [n, k]^T (+ bias [n]) (+ residual [rows, n])
     Tensor linear(const Rows& x, const Tensor& weight, const Tensor* bias = nullptr, const Tensor* residual = nullptr,

@@ -130,6 +130,7 @@ struct CacheRequest {
     int n_kv_heads = 0, head_dim = 0, window = 0;    // KV: keys and values for every position, or the last `window`
     int v_head_dim = 0;                              // KV: size of a value head (0: the keys')
     int keep_first = 0;                              // KV with a window: positions below this stay visible (and held) for good
+    int chunk = 0;                                   // KV: a position sees its own run of this many positions only (0: no such runs; no window then)
     // KV: one row for every `every` positions instead of one per position (row r belongs to positions r * every ..
     // r * every + every - 1: what a mixer keeps of blocks of tokens); such rows have no window
     int every = 1;
@@ -158,6 +159,7 @@ struct CacheView {
     int pool_pages = 0;
     const int* block_table = nullptr;      // [n_seqs][table_width], -1 where the sequence holds no page
     int table_width = 0, page_size = 0, window = 0, n_kv_heads = 0, head_dim = 0;
+    int chunk = 0;                         // CacheRequest::chunk
     int v_head_dim = 0, keep_first = 0;    // values [pages][page_size][kv heads][v_head_dim]; see CacheRequest
     int every = 1;                         // positions per row (CacheRequest::every)
     DType dtype = DType::F32;
@@ -183,6 +185,7 @@ struct StepContext {
     int rows = 0, n_seqs = 0, max_q_len = 0, max_kv_len = 0;
     bool decode = false;                   // every sequence brings exactly one token
     std::vector<int> slots, q_lens, kv_lens;                 // host: per sequence
+    std::vector<int> host_tokens;          // host: the rows' token ids where the step got them from the host (else empty)
     // device, int32: per row, then per sequence
     const int* tokens = nullptr;
     const int* row_seq = nullptr;          // sequence of the step that a row belongs to (negative: a dead row)
@@ -201,6 +204,7 @@ struct BuildEnv {
 struct ParamDecl {
     std::vector<int64_t> shape;     // -1: a size that the checkpoint gives (random weights need every size)
     bool integer = false;    // kept as int32; otherwise in the activation dtype unless stored in 32-bit
+    int64_t below = 0;       // integer: random-weights mode draws the entries of a row, all different, from 0 .. below - 1 (0: zeros)
     bool one = false;        // random-weights mode: 1 + N(0, 0.02) (norm weights) instead of N(0, 0.02)
     // A parameter may be loaded straight into rows of a larger tensor that the part declared with
     // declare_stacked (q, k and v under one another; gate and up row by row in turn): row r of the parameter

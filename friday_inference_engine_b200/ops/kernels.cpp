@@ -121,13 +121,16 @@ FAMILY(Routed, routed, "routed", resolve(h, fam, "routed_route", t.route);
        resolve(h, fam, "routed_down_scratch_floats", t.down_scratch_floats);
        resolve(h, fam, "routed_sort_pairs", t.sort_pairs); resolve(h, fam, "routed_combine", t.combine);
        resolve(h, fam, "routed_route_scored", t.route_scored); resolve(h, fam, "routed_route_biased", t.route_biased);
-       resolve(h, fam, "routed_shared_and_self", t.shared_and_self);)
+       resolve(h, fam, "routed_shared_and_self", t.shared_and_self); resolve(h, fam, "routed_route_table", t.route_table);)
 FAMILY(AttentionTalk, attention_talk, "attention_talk", resolve(h, fam, "attention_talk_store", t.store);
        resolve(h, fam, "attention_talk_scratch_floats", t.scratch_floats); resolve(h, fam, "attention_talk_rows", t.rows);
        resolve(h, fam, "attention_talk_prompt_scratch_floats", t.prompt_scratch_floats);
        resolve(h, fam, "attention_talk_prompt", t.prompt);)
 FAMILY(LinearDecay, linear_decay, "linear_decay", resolve(h, fam, "linear_decay_scratch_floats", t.scratch_floats);
        resolve(h, fam, "linear_decay_run", t.run); resolve(h, fam, "linear_decay_row_norm_gate", t.row_norm_gate);)
+FAMILY(ShortConv, short_conv, "short_conv", resolve(h, fam, "short_conv_heads", t.heads); resolve(h, fam, "short_conv_rows", t.rows);)
+FAMILY(Ssd, ssd, "ssd", resolve(h, fam, "ssd_scratch_floats", t.scratch_floats); resolve(h, fam, "ssd_run", t.run);
+       resolve(h, fam, "ssd_gate_group_norm", t.gate_group_norm);)
 FAMILY(Delta, delta, "delta", resolve(h, fam, "delta_conv_prepare", t.conv_prepare);
        resolve(h, fam, "delta_conv_state", t.conv_state); resolve(h, fam, "delta_scan", t.scan);
        resolve(h, fam, "delta_general_prepare", t.general_prepare); resolve(h, fam, "delta_general_scan", t.general_scan);)

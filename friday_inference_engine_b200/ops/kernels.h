@@ -102,6 +102,20 @@ struct LinearDecay {
                int, int, int, float*, int, cudaStream_t);
     int (*row_norm_gate)(const float*, const void*, int, void*, const void*, int, int, int, float, int, cudaStream_t);
 };
+struct ShortConv {
+    last_error_fn last_error;
+    int (*heads)(const void*, int, int, const void*, int, int, const float*, int, int, float, void*, void*, void*, const int*, int, int, float*, long long,
+                 long long, const int*, const int*, const int*, const int*, const int*, int, int, int, int, int, int, int, int, cudaStream_t);
+    int (*rows)(const void*, int, int, int, const void*, int, int, const void*, int, void*, float*, long long, long long, const int*, const int*,
+                const int*, const int*, int, int, int, int, int, cudaStream_t);
+};
+struct Ssd {
+    last_error_fn last_error;
+    long long (*scratch_floats)(int, int, int, int, int, int);
+    int (*run)(const void*, int, int, int, int, const float*, int, const void*, const void*, const void*, int, float*, float*, long long, long long,
+               const int*, const int*, const int*, const int*, int, int, int, int, int, int, float*, int, cudaStream_t);
+    int (*gate_group_norm)(const float*, const void*, int, int, void*, const void*, int, int, int, int, float, int, cudaStream_t);
+};
 struct Delta {
     last_error_fn last_error;
     int (*conv_prepare)(const void*, int, int, int, int, const void*, int, float*, const float*, long long, const int*, const int*,
@@ -123,12 +137,12 @@ struct AttentionPooled {
                 int, int, int, cudaStream_t);
     long long (*scratch_floats)(int, int, int, int);
     int (*rows)(const void*, int, int, void*, const void*, const void*, const float*, const float*, const int*, int, const int*, int, int,
-                const int*, const int*, int, int, int, int, int, int, int, float, float, int, float, const void*, int, const void*, int, float*,
-                int, cudaStream_t);
+                const int*, const int*, int, int, int, int, int, int, int, float, float, int, float, const void*, int, const void*, int, int, int, int,
+                float*, int, cudaStream_t);
     int (*prompt_fits)(int, int, int);
     int (*prompt)(const void*, int, int, void*, const void*, const void*, const float*, const float*, const int*, int, const int*, int, int,
                   const int*, const int*, const int*, int, int, int, int, int, int, int, int, float, float, int, float, const void*, int,
-                  const void*, cudaStream_t);
+                  const void*, int, int, int, cudaStream_t);
 };
 struct AttentionLatent {
     last_error_fn last_error;
@@ -156,6 +170,7 @@ struct Routed {
     int (*combine)(const float*, const int*, const float*, const int*, const void*, void*, int, int, int, int, cudaStream_t);
     int (*route_scored)(const float*, int, int, int, int, const void*, int, int, int, float, int*, float*, float*, cudaStream_t);
     int (*route_biased)(const float*, int, int, int, int, int, const void*, int, int*, float*, float*, float*, cudaStream_t);
+    int (*route_table)(const int*, const int*, int, int, int, int, int*, float*, float*, cudaStream_t);
     int (*shared_and_self)(const float*, const float*, const float*, int, const float*, const void*, float*, int, int, int, cudaStream_t);
 };
 struct AttentionTalk {
@@ -176,14 +191,14 @@ struct AttentionMma {
                cudaStream_t);
     int (*clusters_at_once)(int, int);
     int (*extra)(const void*, int, void*, const void*, const void*, int, const int*, int, int, const int*, const int*, const int*, const int*, int,
-                 int, int, int, int, int, float, float, const void*, int, const void*, int, float*, int*, int, int*, cudaStream_t);
+                 int, int, int, int, int, float, float, const void*, int, const void*, int, int, int, int, float*, int*, int, int*, cudaStream_t);
 };
 struct AttentionTc {
     last_error_fn last_error;
     int (*run)(const void*, int, int, void*, const void*, const void*, int, const int*, int, const int*, const int*,
                const int*, const int*, int, int, int, int, int, int, float, int*, cudaStream_t);
     int (*extra)(const void*, int, int, void*, const void*, const void*, int, const int*, int, const int*, const int*, const int*, const int*, int,
-                 int, int, int, int, int, int, float, float, const void*, int, const void*, int, int*, cudaStream_t);
+                 int, int, int, int, int, int, float, float, const void*, int, const void*, int, int, int, int*, cudaStream_t);
 };
 struct Sampling {
     last_error_fn last_error;
@@ -203,6 +218,8 @@ const Residual& residual();
 const Recurrence& recurrence();
 const Routed& routed();
 const LinearDecay& linear_decay();
+const ShortConv& short_conv();
+const Ssd& ssd();
 const Delta& delta();
 const AttentionLatent& attention_latent();
 const AttentionTalk& attention_talk();

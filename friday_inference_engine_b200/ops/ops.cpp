@@ -559,7 +559,13 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
     check_pooled(s, tokens, pooled, proj.dtype);
     const auto& k = kernels::attention_pooled();
     Tensor out = alloc(proj.dtype, proj.rows(), (int64_t)s.heads * s.vdim);
-    const void* gate = s.gate_off >= 0 ? (const char*)proj.data + (size_t)s.gate_off * dtype_size(proj.dtype) : nullptr;
+    const Tensor& gates = s.gate_rows ? *s.gate_rows : proj;
+    if (gates.dtype != proj.dtype || gates.rows() != proj.rows()) throw KernelError("pooled attention: the gates are rows of the queries' number and dtype");
+    const void* gate = s.gate_off >= 0 ? (const char*)gates.data + (size_t)s.gate_off * dtype_size(proj.dtype) : nullptr;
+    const int gate_ld = (int)gates.ld, wide = s.gate_wide ? 1 : 0;
+    if (s.chunk < 0 || (s.chunk > 0 && (s.window > 0 || s.pool > 0)) || s.chunk != tokens.chunk)
+        throw KernelError("pooled attention: runs of positions go without a window, and the cache holds what they need");
+    const bool gates_ok = !gate || !wide || (gate_ld % 8 == 0 && s.gate_off % 8 == 0 && s.vdim % 8 == 0 && aligned16(gate));
     const float* pk = pooled ? (const float*)pooled->k_pool : nullptr;
     const float* pv = pooled ? (const float*)pooled->v_pool : nullptr;
     const int* ptable = pooled ? pooled->block_table : nullptr;
@@ -568,14 +574,14 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
     // FRIDAY_POOLED_TCGEN05=0 leaves them to the kernel below
     const bool tcgen05 = proj.dtype == DType::BF16 && !ctx.decode && ctx.max_q_len >= 16 && s.pool == 0 && s.temp_every == 0 && s.v_off >= 0 &&
                          attn_tc_ && env_on("FRIDAY_POOLED_TCGEN05") && s.dim % 16 == 0 && s.dim <= 128 && s.vdim % 16 == 0 && s.vdim <= 128 &&
-                         tokens.page_size == 64 && s.heads / s.kv_heads <= 128 && proj.ld % 8 == 0 && s.q_off % 8 == 0 && aligned16(proj.data);
+                         gates_ok && tokens.page_size == 64 && s.heads / s.kv_heads <= 128 && proj.ld % 8 == 0 && s.q_off % 8 == 0 && aligned16(proj.data);
     if (tcgen05) {
         const auto& a = kernels::attention_tc();
         Timed t(*this, Attention);
         call(launches_, a, a.extra((const char*)proj.data + (size_t)s.q_off * dtype_size(proj.dtype), (int)proj.ld, (int)proj.rows(), out.data, tokens.k_pool,
                                    tokens.v_pool, tokens.pool_pages, tokens.block_table, tokens.table_width, ctx.seq_start, ctx.seq_qlen, ctx.seq_pos0,
                                    ctx.row_seq, ctx.n_seqs, ctx.max_q_len, s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.scale, s.softcap,
-                                   s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, (int)proj.ld, (int*)status_.get(), stream_),
+                                   s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, gate_ld, wide, s.chunk, (int*)status_.get(), stream_),
              "attention_tc_extra");
         return out;
     }
@@ -583,17 +589,17 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
     // shares a sequence's keys among CTAs (FRIDAY_POOLED_MMA=0: the CUDA-core kernel)
     const int64_t counters_needed = (int64_t)ctx.n_seqs * s.kv_heads * ((s.heads / s.kv_heads + 15) / 16);
     if (proj.dtype == DType::BF16 && ctx.decode && ctx.seq_start != nullptr && s.pool == 0 && s.temp_every == 0 && s.v_off >= 0 && s.vdim == s.dim &&
-        env_on("FRIDAY_POOLED_MMA") && s.dim % 16 == 0 && s.dim <= 128 && tokens.page_size == 64 && proj.ld % 8 == 0 && s.q_off % 8 == 0 &&
+        gates_ok && env_on("FRIDAY_POOLED_MMA") && s.dim % 16 == 0 && s.dim <= 128 && tokens.page_size == 64 && proj.ld % 8 == 0 && s.q_off % 8 == 0 &&
         aligned16(proj.data) && (int)proj.rows() == ctx.n_seqs && counters_needed <= (int64_t)(attn_counters_.bytes() / sizeof(int)) &&
         s.kv_heads <= 65535 && ctx.n_seqs <= 65535) {
-        const int splits = decode_splits(ctx.n_seqs, s.heads, s.kv_heads, s.dim, ctx.max_kv_len);
+        const int splits = decode_splits(ctx.n_seqs, s.heads, s.kv_heads, s.dim, s.chunk > 0 ? std::min(ctx.max_kv_len, s.chunk) : ctx.max_kv_len);
         float* scratch = splits > 1 ? scratch_floats(proj.rows() * s.heads * splits * (s.dim + 2)) : nullptr;
         const auto& a = kernels::attention_mma();
         Timed t(*this, Attention);
         call(launches_, a, a.extra((const char*)proj.data + (size_t)s.q_off * dtype_size(proj.dtype), (int)proj.ld, out.data, tokens.k_pool, tokens.v_pool,
                                    tokens.pool_pages, tokens.block_table, tokens.table_width, 64, ctx.seq_start, ctx.seq_qlen, ctx.seq_pos0, ctx.row_seq,
                                    ctx.n_seqs, (int)proj.rows(), s.heads, s.kv_heads, s.dim, s.window, s.scale, s.softcap,
-                                   s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, splits, scratch,
+                                   s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, gate_ld, wide, s.chunk, splits, scratch,
                                    (int*)attn_counters_.get(), (int)(attn_counters_.bytes() / sizeof(int)), (int*)status_.get(), stream_),
              "attention_mma_extra");
         return out;
@@ -605,19 +611,91 @@ Tensor Ops::pooled_attention(const Tensor& proj, const PooledSpec& s, const Cach
         call(launches_, k, k.prompt(proj.data, (int)proj.ld, (int)s.q_off, out.data, tokens.k_pool, tokens.v_pool, pk, pv, tokens.block_table,
                                     tokens.table_width, ptable, pwidth, tokens.page_size, ctx.seq_start, ctx.seq_qlen, ctx.seq_pos0, ctx.n_seqs,
                                     ctx.max_q_len, s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.pool, s.scale, s.temp_coef, s.temp_every, s.softcap,
-                                    s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, stream_), "pooled prompt");
+                                    s.sink ? s.sink->data : nullptr, s.sink ? code(s.sink->dtype) : 0, gate, gate_ld, wide, s.chunk, stream_), "pooled prompt");
         return out;
     }
     // keys that a row can face: its window (or everything before it) and the pooled blocks
     int keys = ctx.max_kv_len;
+    if (s.chunk > 0) keys = std::min(keys, s.chunk);
     if (s.window > 0) keys = std::min(keys, s.window + (s.pool > 0 ? ctx.max_kv_len / s.pool : 0));
     const int splits = attention_splits(proj.rows(), s.heads, keys);
     float* scratch = scratch_floats(k.scratch_floats((int)proj.rows(), s.heads, s.vdim, splits));
     call(launches_, k, k.rows(proj.data, (int)proj.ld, (int)s.q_off, out.data, tokens.k_pool, tokens.v_pool, pk, pv, tokens.block_table,
                               tokens.table_width, ptable, pwidth, tokens.page_size, ctx.row_seq, ctx.row_pos, (int)proj.rows(), s.heads, s.kv_heads,
                               s.dim, s.vdim, s.window, s.pool, s.scale, s.temp_coef, s.temp_every, s.softcap, s.sink ? s.sink->data : nullptr,
-                              s.sink ? code(s.sink->dtype) : 0, gate, splits, scratch, code(proj.dtype), stream_), "pooled rows");
+                              s.sink ? code(s.sink->dtype) : 0, gate, gate_ld, wide, s.chunk, splits, scratch, code(proj.dtype), stream_), "pooled rows");
     ++launches_;                                     // the merge
+    return out;
+}
+
+// ------------------------------------------------------------------ short convolutions, state space duality
+static long long check_conv(const Tensor& proj, int64_t off, int64_t channels, const Tensor& taps, const CacheView& state, int64_t hist_off) {
+    if (state.kind != CacheRequest::State || !state.state.defined() || state.state.dtype != DType::F32) throw KernelError("a short convolution needs a 32-bit state view");
+    const long long stride = state.state.numel() / state.state.shape[0];
+    if (taps.ndim != 2 || !taps.contiguous() || taps.rows() != channels || off < 0 || off + channels > proj.cols() || hist_off + (taps.cols() - 1) * channels > stride)
+        throw KernelError("a short convolution: taps [channels, n], that many columns of the rows, and a state that holds n - 1 inputs");
+    return stride;
+}
+
+Tensor Ops::conv_heads(const Tensor& proj, const Tensor& taps, const ConvSpec& s, const CacheView& tokens, const CacheView& state, const StepContext& ctx) {
+    if (tokens.kind != CacheRequest::KV || !tokens.k_pool || !tokens.write || tokens.dtype != proj.dtype || tokens.n_kv_heads != s.kv_heads ||
+        tokens.head_dim != s.dim || (tokens.v_head_dim > 0 ? tokens.v_head_dim : tokens.head_dim) != s.vdim || tokens.every != 1)
+        throw KernelError("conv_heads: the cache view does not hold this mixer's keys and values in the rows' dtype");
+    const long long stride = check_conv(proj, s.off, (int64_t)(s.heads + s.kv_heads) * s.dim + (int64_t)s.kv_heads * s.vdim, taps, state, s.hist_off);
+    Tensor q = alloc(proj.dtype, proj.rows(), (int64_t)s.heads * s.dim);
+    const auto& k = kernels::short_conv();
+    Timed t(*this, Other);
+    call(launches_, k, k.heads(proj.data, (int)proj.ld, (int)s.off, taps.data, code(taps.dtype), (int)taps.cols(), s.freq, s.rot, s.unit_norm ? 1 : 0, s.eps,
+                               q.data, tokens.k_pool, tokens.v_pool, tokens.block_table, tokens.table_width, tokens.page_size, (float*)state.state.data,
+                               stride, s.hist_off, ctx.row_seq, ctx.row_pos, ctx.seq_start, ctx.seq_qlen, state.seq_slots, ctx.n_seqs, (int)proj.rows(),
+                               s.heads, s.kv_heads, s.dim, s.vdim, ctx.decode ? 1 : 0, code(proj.dtype), stream_), "conv_heads");
+    if (!ctx.decode && taps.cols() > 1) ++launches_;         // the history
+    return q;
+}
+
+Tensor Ops::conv_silu_rows(const Tensor& proj, int64_t off, int64_t channels, const Tensor& taps, const Tensor* bias, const CacheView& state, int64_t hist_off,
+                           DType dtype, const StepContext& ctx) {
+    const long long stride = check_conv(proj, off, channels, taps, state, hist_off);
+    if (bias && bias->numel() != channels) throw KernelError("conv_silu_rows: a bias per channel");
+    Tensor out = alloc(dtype, proj.rows(), channels);
+    const auto& k = kernels::short_conv();
+    Timed t(*this, Other);
+    call(launches_, k, k.rows(proj.data, (int)proj.ld, (int)off, (int)channels, taps.data, code(taps.dtype), (int)taps.cols(), bias ? bias->data : nullptr,
+                              bias ? code(bias->dtype) : 0, out.data, (float*)state.state.data, stride, hist_off, ctx.row_seq, ctx.seq_start, ctx.seq_qlen,
+                              state.seq_slots, ctx.n_seqs, (int)proj.rows(), ctx.decode ? 1 : 0, code(proj.dtype), code(dtype), stream_), "conv_silu_rows");
+    if (!ctx.decode && taps.cols() > 1) ++launches_;         // the history
+    return out;
+}
+
+Tensor Ops::ssd_scan(const Tensor& xbc, const Tensor& dt, const Tensor& dt_bias, const Tensor& a_log, const Tensor& skip, const SsdSpec& s,
+                     const CacheView& view, const StepContext& ctx) {
+    if (view.kind != CacheRequest::State || !view.state.defined() || view.state.dtype != DType::F32) throw KernelError("ssd_scan needs a 32-bit state view");
+    if (dt.dtype != DType::F32 || dt.rows() != xbc.rows() || dt.cols() < s.heads) throw KernelError("ssd_scan: 32-bit step sizes, one per row and head");
+    if (dt_bias.numel() != s.heads || a_log.numel() != s.heads || skip.numel() != s.heads || dt_bias.dtype != a_log.dtype || dt_bias.dtype != skip.dtype)
+        throw KernelError("ssd_scan: a bias, a decay rate and a skip weight per head, of one dtype");
+    const long long stride = view.state.numel() / view.state.shape[0];
+    Tensor out = alloc(DType::F32, xbc.rows(), (int64_t)s.heads * s.vdim);
+    const auto& k = kernels::ssd();
+    // FRIDAY_SSD_CHUNKS=0 keeps prompts on the token-by-token kernel (for comparisons)
+    const long long need = !ctx.decode && env_on("FRIDAY_SSD_CHUNKS") ? k.scratch_floats(ctx.n_seqs, ctx.max_q_len, s.heads, s.state, s.vdim, code(xbc.dtype)) : 0;
+    float* scratch = need > 0 ? scratch_floats(need) : nullptr;
+    Timed t(*this, Attention);
+    call(launches_, k, k.run(xbc.data, (int)xbc.ld, (int)s.x_off, (int)s.b_off, (int)s.c_off, (const float*)dt.data, (int)dt.ld, dt_bias.data, a_log.data,
+                             skip.data, code(dt_bias.dtype), (float*)out.data, (float*)view.state.data, stride, s.s_off, ctx.row_seq, ctx.seq_start,
+                             ctx.seq_qlen, view.seq_slots, ctx.n_seqs, ctx.max_q_len, s.heads, s.groups, s.state, s.vdim, scratch, code(xbc.dtype), stream_),
+         "ssd");
+    if (scratch) launches_ += 2;
+    return out;
+}
+
+Tensor Ops::gate_group_norm(const Tensor& y, const Tensor& z, const Tensor& weight, int parts, float eps, DType dtype) {
+    if (y.dtype != DType::F32 || !y.contiguous() || z.rows() != y.rows() || z.cols() != y.cols() || weight.numel() != y.cols())
+        throw KernelError("gate_group_norm: fp32 rows, a gate of their size, a weight per channel");
+    Tensor out = alloc(dtype, y.rows(), y.cols());
+    const auto& k = kernels::ssd();
+    Timed t(*this, Other);
+    call(launches_, k, k.gate_group_norm((const float*)y.data, z.data, (int)z.ld, code(z.dtype), out.data, weight.data, code(weight.dtype), (int)y.rows(),
+                                         (int)y.cols(), parts, eps, code(dtype), stream_), "gate_group_norm");
     return out;
 }
 
@@ -911,6 +989,20 @@ Ops::Routing Ops::route_biased(const Tensor& logits, int experts, int identity, 
     return r;
 }
 
+Ops::Routing Ops::route_table(const int* tokens, int64_t rows, const Tensor& table, int experts, bool with_dense) {
+    if (table.dtype != DType::I32 || table.ndim != 2 || !table.contiguous()) throw KernelError("route: a table [vocab, choices] of integers");
+    Routing r;
+    const int64_t top = table.cols();
+    r.ids = Tensor::make(arena->alloc((size_t)rows * top * sizeof(int)), DType::I32, {rows, top});
+    r.weights = alloc(DType::F32, rows, top);
+    if (with_dense) r.dense = alloc(DType::F32, rows, experts);
+    const auto& k = kernels::routed();
+    Timed t(*this, Other);
+    call(launches_, k, k.route_table(tokens, (const int*)table.data, (int)table.rows(), (int)rows, experts, (int)top, (int*)r.ids.data,
+                                     (float*)r.weights.data, with_dense ? (float*)r.dense.data : nullptr, stream_), "route_table");
+    return r;
+}
+
 Tensor Ops::shared_and_self(const Tensor* residual, const Tensor* shared, const Tensor* logits, int64_t gate_col, const Tensor* self, const Tensor& h) {
     for (const Tensor* t : {residual, shared})
         if (t && (t->dtype != DType::F32 || !t->contiguous() || t->numel() != h.numel())) throw KernelError("shared_and_self: contiguous 32-bit rows of the input's size");
@@ -961,7 +1053,7 @@ Tensor Ops::expert_down_combine(const Tensor& act, const Routing& r, const Tenso
 }
 
 Tensor Ops::experts_grouped(const Tensor& h, const Routing& r, const Tensor& w_gate_up, const Tensor& w_down, const Tensor& residual,
-                            int top, int inner, int unit, float limit, float slope) {
+                            int top, int inner, int unit, float limit, float slope, const std::vector<int>* counts) {
     const int64_t rows = h.rows(), width = h.cols(), n_pairs = rows * top;
     const int experts = (int)(w_gate_up.rows() / (2 * (int64_t)inner));
     const auto& k = kernels::routed();
@@ -973,8 +1065,13 @@ Tensor Ops::experts_grouped(const Tensor& h, const Routing& r, const Tensor& w_g
         call(launches_, k, k.sort_pairs((const int*)r.ids.data, (int)rows, top, experts, offsets, pos, row_at, stream_), "sort_pairs");
     }
     std::vector<int> off((size_t)experts + 1);
-    cuda_check(cudaMemcpyAsync(off.data(), offsets, off.size() * sizeof(int), cudaMemcpyDeviceToHost, stream_), "cudaMemcpyAsync");
-    cuda_check(cudaStreamSynchronize(stream_), "cudaStreamSynchronize");
+    if (counts) {
+        if ((int)counts->size() != experts) throw KernelError("experts_grouped: a number of choices per expert");
+        for (int e = 0; e < experts; ++e) off[(size_t)e + 1] = off[(size_t)e] + (*counts)[(size_t)e];
+    } else {
+        cuda_check(cudaMemcpyAsync(off.data(), offsets, off.size() * sizeof(int), cudaMemcpyDeviceToHost, stream_), "cudaMemcpyAsync");
+        cuda_check(cudaStreamSynchronize(stream_), "cudaStreamSynchronize");
+    }
     // (fewer places than pairs where some choices are no expert of this table: only the places that exist are gathered)
     Tensor gathered = off.back() > 0 ? gather_rows(row_at, off.back(), h) : Tensor();
     Tensor part = alloc(DType::F32, n_pairs, width);

@@ -607,6 +607,7 @@ public:
         Tensor inner = ops.linear_swiglu(h, tensor("w_gate_up"), act_);
         Tensor nw;
         float eps;
+        if (!residual.defined()) return PartOut(ops.linear(Rows(inner), tensor(down_), nullptr, nullptr, (int)DType::F32));     // the block sums itself
         if (then && residual.dtype == inner.dtype && then->as_rmsnorm(&nw, &eps)) {
             auto r = ops.linear_norm(Rows(inner), tensor(down_), nw, eps, nullptr, &residual);
             return PartOut(r.first, r.second);

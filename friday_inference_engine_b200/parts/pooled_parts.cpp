@@ -14,7 +14,12 @@
 //                              "v.b"); "qk_norm": "whole" norms all query heads of a row at once (weights [heads * dim]),
 //                              likewise the keys; "softcap" c: score <- c tanh(score / c); "head_gate": head h's result is
 //                              multiplied by sigmoid(Wg h)_h (tensor "g" [heads, width]); "shared_kv": no keys and values of its
-//                              own (nor their norm), it reads the cache entry of an earlier layer.
+//                              own (nor their norm), it reads the cache entry of an earlier layer; "conv" n: q, k and v as projected pass a
+//                              causal convolution over time with n taps per channel (tensors "q.conv", "k.conv", "v.conv" [channels, n], zeros
+//                              before a sequence's start, the last n - 1 inputs in its state) ahead of everything else; "qk_norm": "unit"
+//                              divides every q and k head by its root mean square AFTER the rotation, without a weight (goes with a
+//                              convolution); "gate": the concatenated heads are multiplied element by element by sigmoid(Wg h) (tensor "g"
+//                              [heads * vdim, width]); "chunk" C: row i sees token j <= i if floor(i / C) = floor(j / C).
 //   mixer "general_delta"      r, k, v = W h (heads x dim); decay w = exp(-rate * sigmoid(Ww2 tanh(Ww1 h) + w0)) and removal
 //                              a = sigmoid(Wa h + a.b) per head and key channel; with the unit key u = k / sqrt(sum k^2 + 1e-6):
 //                              S <- diag(w) S - (a u)(u^T S) + k v^T (both terms read the old S), o = S^T r; every head's o
@@ -25,6 +30,7 @@
 // csrc/delta.cu).  Handed an undefined residual, a mixer returns its result alone as 32-bit rows.
 #include <math.h>
 
+#include <algorithm>
 #include <string>
 
 #include "friday/ops.h"
@@ -73,13 +79,17 @@ public:
         eps_ = (float)s.params.get_double("eps", 1e-5);
         has_sink_ = s.params.get_bool("sink", false);
         const Json* qn = s.params.find("qk_norm");
-        if (qn && !qn->is_bool() && !(qn->is_string() && (qn->as_string() == "heads" || qn->as_string() == "whole")))
-            throw ConfigError("pooled_attention: 'qk_norm' is true, false, \"heads\" or \"whole\"");
+        if (qn && !qn->is_bool() && !(qn->is_string() && (qn->as_string() == "heads" || qn->as_string() == "whole" || qn->as_string() == "unit")))
+            throw ConfigError("pooled_attention: 'qk_norm' is true, false, \"heads\", \"whole\" or \"unit\"");
+        unit_norm_ = qn && qn->is_string() && qn->as_string() == "unit";
         norm_whole_ = qn && qn->is_string() && qn->as_string() == "whole";
-        qk_norm_ = norm_whole_ || (qn && (qn->is_string() || qn->as_bool()));
+        qk_norm_ = !unit_norm_ && (norm_whole_ || (qn && (qn->is_string() || qn->as_bool())));
         softcap_ = (float)s.params.get_double("softcap", 0.0);
         bias_ = s.params.get_bool("qkv_bias", false);
         head_gate_ = s.params.get_bool("head_gate", false);
+        wide_gate_ = s.params.get_bool("gate", false);
+        taps_ = (int)s.params.get_int("conv", 0);
+        chunk_ = (int)s.params.get_int("chunk", 0);
         reads_ = s.params.get_bool("shared_kv", false);
         const std::string values = s.params.get_string("values", "own");
         if (values != "own" && values != "keys") throw ConfigError("pooled_attention: 'values' is \"own\" or \"keys\"");
@@ -91,6 +101,11 @@ public:
         if (reads_ && (shared_ || pool_ > 0)) throw ConfigError("pooled_attention: a layer that reads another's keys and values has values of its own kind and no pooled blocks");
         if (window_ < 0 || pool_ < 0) throw ConfigError("pooled_attention: 'window' and 'pool' must not be negative");
         if (pool_ > 0 && window_ == 0) throw ConfigError("pooled_attention: pooled blocks lie before a window; without a window every token is seen");
+        if (chunk_ < 0 || taps_ < 0) throw ConfigError("pooled_attention: 'chunk' and 'conv' must not be negative");
+        if (chunk_ > 0 && (window_ > 0 || pool_ > 0 || reads_)) throw ConfigError("pooled_attention: runs of positions go without a window, and with keys and values of the layer's own");
+        if (head_gate_ && wide_gate_) throw ConfigError("pooled_attention: a gate per head or a gate per channel");
+        if (taps_ > 0 && (shared_ || reads_ || pool_ > 0 || qk_norm_)) throw ConfigError("pooled_attention: a convolution goes with keys and values of the layer's own, no pooled blocks and no weighted norm of the heads");
+        if (unit_norm_ && taps_ == 0) throw ConfigError("pooled_attention: a norm without a weight after the rotation goes with a convolution (of one tap at least)");
         const Json* qt = s.params.find("q_temp");
         if (qt && qt->is_object()) {
             temp_coef_ = (float)qt->get_double("coef", 0.0);
@@ -99,7 +114,7 @@ public:
         }
         position_ = adopt("", build<Position>("position", s.part("position"), e));
         const int64_t w = e.width, qd = (int64_t)heads_ * dim_, kd = reads_ ? 0 : (int64_t)kv_heads_ * dim_;
-        const int64_t vd = shared_ || reads_ ? 0 : (int64_t)kv_heads_ * vdim_, gd = head_gate_ ? heads_ : 0;
+        const int64_t vd = shared_ || reads_ ? 0 : (int64_t)kv_heads_ * vdim_, gd = wide_gate_ ? (int64_t)heads_ * vdim_ : head_gate_ ? heads_ : 0;
         // one product for queries, keys, values and gates; its columns are padded to whole 16-byte pieces, since the rows' queries
         // and values are read as such
         declare_stacked("w_in", (qd + kd + vd + gd + 7) / 8 * 8, w);
@@ -117,12 +132,23 @@ public:
             declare("q.norm", {norm_whole_ ? qd : (int64_t)dim_}, false, true);
             if (kd) declare("k.norm", {norm_whole_ ? kd : (int64_t)dim_}, false, true);
         }
+        if (taps_ > 0) {
+            declare_stacked("taps", qd + kd + vd, taps_);
+            declare("q.conv", {qd, (int64_t)taps_}).stack("taps", 0);
+            declare("k.conv", {kd, (int64_t)taps_}).stack("taps", qd);
+            declare("v.conv", {vd, (int64_t)taps_}).stack("taps", qd + kd);
+        }
         if (has_sink_) declare("sink", {(int64_t)heads_});
         declare("o", {w, (int64_t)heads_ * vdim_});
     }
     CacheRequest cache_request() const override {
         CacheRequest tokens = CacheRequest::kv(kv_heads_, dim_, window_, vdim_, 0);
         tokens.keys_only = shared_;
+        tokens.chunk = chunk_;
+        if (taps_ > 0) {                                         // beside them the convolution's last inputs
+            const int64_t channels = (int64_t)(heads_ + kv_heads_) * dim_ + (int64_t)kv_heads_ * vdim_;
+            return CacheRequest::several({tokens, CacheRequest::state({std::max<int64_t>(1, (taps_ - 1) * channels)}, DType::F32)});
+        }
         if (pool_ == 0) return tokens;
         CacheRequest blocks = CacheRequest::kv(kv_heads_, dim_, 0, vdim_, 0);
         blocks.every = pool_;
@@ -137,6 +163,7 @@ public:
         neighbours_ = position_->pairs(&freq_, &rot_mult_, &rot_);
         if (neighbours_ || position_->halves(&freq_, &rot_mult_, &rot_)) {
             if (rot_ > dim_ || rot_ % 2) throw ConfigError(format("%s: %d rotated numbers in heads of %d", prefix.c_str(), rot_, dim_));
+            if (taps_ > 0 && (!neighbours_ || rot_mult_ != 1.0f)) throw ConfigError(prefix + ": a convolution goes with plainly rotated neighbouring pairs, or no rotation");
             if (norm_whole_ && !neighbours_) throw ConfigError(prefix + ": a norm over all heads at once goes with neighbouring pairs, or no rotation");
         } else if (position_->rotary(&denominators, &d)) {
             throw ConfigError(prefix + ": pooled_attention takes a position part with a table of frequencies, or none");
@@ -146,10 +173,10 @@ public:
     PartOut forward(Ops& ops, const Rows& h, const Tensor& residual, const StepContext& ctx, const CacheView& view, Norm*) override {
         const CacheView* tokens = &view;
         const CacheView* blocks = nullptr;
-        if (pool_ > 0) {
-            if (view.kind != CacheRequest::Several || view.parts.size() != 2) throw KernelError("pooled_attention: the cache view lacks the tokens' part or the blocks'");
+        if (pool_ > 0 || taps_ > 0) {
+            if (view.kind != CacheRequest::Several || view.parts.size() != 2) throw KernelError("pooled_attention: the cache view lacks the tokens' part, or the blocks' or the convolution's");
             tokens = &view.parts[0];
-            blocks = &view.parts[1];
+            if (pool_ > 0) blocks = &view.parts[1];
         }
         Tensor bias_flat;
         if (bias_) {
@@ -181,7 +208,24 @@ public:
         sp.q_off = 0;
         sp.k_off = reads_ ? -1 : qd;
         sp.v_off = shared_ ? -1 : qd + kd;
-        sp.gate_off = head_gate_ ? qd + kd + vd : -1;
+        sp.gate_off = head_gate_ || wide_gate_ ? qd + kd + vd : -1;
+        sp.gate_wide = wide_gate_;
+        sp.chunk = chunk_;
+        if (taps_ > 0) {                                         // the queries leave the projection's rows, which the convolution still reads
+            Ops::ConvSpec cs;
+            cs.heads = heads_;
+            cs.kv_heads = kv_heads_;
+            cs.dim = dim_;
+            cs.vdim = vdim_;
+            cs.freq = freq_;
+            cs.rot = rot_;
+            cs.unit_norm = unit_norm_;
+            cs.eps = eps_;
+            Tensor q = ops.conv_heads(in, tensor("taps"), cs, *tokens, view.parts[1], ctx);
+            sp.gate_rows = &in;
+            Tensor mixed = ops.pooled_attention(q, sp, *tokens, nullptr, ctx);
+            return project_out(ops, mixed, tensor("o"), residual, out_scale);
+        }
         ops.pooled_store(in, sp, *tokens, blocks, ctx);
         Tensor mixed = ops.pooled_attention(in, sp, *tokens, blocks, ctx);
         return project_out(ops, mixed, tensor("o"), residual, out_scale);
@@ -190,7 +234,8 @@ public:
 private:
     int heads_, kv_heads_, dim_, vdim_, window_, pool_, temp_every_ = 0, rot_ = 0;
     float scale_, eps_, temp_coef_ = 0.f, rot_mult_ = 1.0f, softcap_ = 0.f;
-    bool has_sink_, qk_norm_, shared_, norm_whole_ = false, bias_ = false, head_gate_ = false, reads_ = false, neighbours_ = false;
+    bool has_sink_, qk_norm_, shared_, norm_whole_ = false, bias_ = false, head_gate_ = false, reads_ = false, neighbours_ = false, unit_norm_ = false, wide_gate_ = false;
+    int taps_ = 0, chunk_ = 0;
     Position* position_;
     const float* freq_ = nullptr;
 };

@@ -10,7 +10,9 @@
 //                                    entry part of its own
 //   feed_forward "routed_experts"    top-k of a biased router, weights by softmax over the chosen logits, gated experts; or
 //                                    sigmoid scores with a choice bias and groups of experts, or softmax scores with a choice bias
-//                                    and experts that return their input; and an expert for every row
+//                                    and experts that return their input; or a table of the token ids; and an expert for every row
+//   mixer "state_space_dual"         S_t = exp(-exp(A) dt_t) S_(t-1) + dt_t B_t x_t^T,  y_t = S_t^T C_t + D x_t, x, B and C through a short
+//                                    convolution and silu
 //   token_input "gated_token_table"  x += norm(proj(gelu_tanh(gate x) * table[token]))
 //
 // The states, the decays and everything that enters the recurrences besides the projections are fp32 (csrc/recurrence.cu);
@@ -19,6 +21,7 @@
 #include <math.h>
 #include <stdlib.h>
 
+#include <algorithm>
 #include <string>
 
 #include "friday/ops.h"
@@ -233,6 +236,82 @@ private:
     float eps_;
 };
 
+// ------------------------------------------------------------------ state space duality
+// W_in h = [z (heads x vdim) | x (heads x vdim) | B (groups x state) | C (groups x state) | dt (heads)]; x, B and C pass a causal convolution per
+// channel ("conv" taps, with a bias, zeros before a sequence's start) and silu; dt = softplus(dt + dt_bias); per head (group h / (heads / groups))
+// S = exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x; the heads' results side by side times silu(z), each of "norm_groups" equal runs of the
+// row divided by its own root mean square, times the weight "norm", then Wo.  State per sequence, fp32: the convolution's last taps - 1 inputs,
+// then the heads' matrices.
+class StateSpaceDual : public Mixer {
+public:
+    StateSpaceDual(const PartSpec& s, const BuildEnv& e) : Mixer(e) {
+        heads_ = positive(s, "heads", "state_space_dual");
+        vdim_ = positive(s, "vdim", "state_space_dual");
+        n_ = positive(s, "state", "state_space_dual");
+        groups_ = positive(s, "groups", "state_space_dual");
+        taps_ = positive(s, "conv", "state_space_dual");
+        norm_groups_ = (int)s.params.get_int("norm_groups", 1);
+        eps_ = (float)s.params.get_double("eps", 1e-5);
+        if (heads_ % groups_) throw ConfigError(format("state_space_dual: %d heads cannot share %d groups", heads_, groups_));
+        if (n_ > 512) throw ConfigError("state_space_dual: at most 512 rows of state per head");
+        inner_ = (int64_t)heads_ * vdim_;
+        gn_ = (int64_t)groups_ * n_;
+        if (norm_groups_ < 1 || inner_ % norm_groups_) throw ConfigError(format("state_space_dual: a norm over %lld channels in %d equal parts", (long long)inner_, norm_groups_));
+        const int64_t w = e.width;
+        declare("in", {2 * inner_ + 2 * gn_ + heads_, w});
+        declare("conv", {inner_ + 2 * gn_, (int64_t)taps_});
+        declare("conv.b", {inner_ + 2 * gn_});
+        // three numbers per head, kept together so that they have one dtype
+        declare_stacked("per_head", 3 * (int64_t)heads_, 1);
+        declare("dt_bias", {(int64_t)heads_}).stack("per_head", 0);
+        declare("A_log", {(int64_t)heads_}).stack("per_head", heads_);
+        declare("D", {(int64_t)heads_}).stack("per_head", 2 * (int64_t)heads_);
+        declare("norm", {inner_}, false, true);
+        declare("o", {w, inner_});
+    }
+    CacheRequest cache_request() const override {
+        return CacheRequest::state({(int64_t)(taps_ - 1) * (inner_ + 2 * gn_) + (int64_t)heads_ * n_ * vdim_}, DType::F32);
+    }
+
+    PartOut forward(Ops& ops, const Rows& h, const Tensor& residual, const StepContext& ctx, const CacheView& view, Norm*) override {
+        const Tensor& w_in = tensor("in");
+        const int64_t main = 2 * inner_ + 2 * gn_, all = main + heads_;
+        Tensor x = ops.materialize(h), in, dt;
+        if (x.dtype == DType::F32 || x.rows() <= 64) {
+            in = ops.linear(Rows(x), w_in, nullptr, nullptr, (int)DType::F32);
+            dt = columns(in, main, heads_);
+        } else {
+            // many rows: everything but the step sizes in the activation dtype (rows of whole 16-byte pieces, where the matrix has them)
+            in = ops.linear(Rows(x), w_in.row_slice(0, std::min((main + 7) / 8 * 8, all)));
+            dt = ops.linear(Rows(x), w_in.row_slice(main, heads_), nullptr, nullptr, (int)DType::F32);
+        }
+        const Tensor& taps = tensor("conv");
+        Tensor xbc = ops.conv_silu_rows(in, inner_, inner_ + 2 * gn_, taps, &tensor("conv.b"), view, 0, x.dtype, ctx);
+        const Tensor& ph = tensor("per_head");
+        auto head_vector = [&](int64_t i) { return Tensor::make((char*)ph.data + (size_t)i * heads_ * dtype_size(ph.dtype), ph.dtype, {(int64_t)heads_}); };
+        Ops::SsdSpec sp;
+        sp.heads = heads_;
+        sp.groups = groups_;
+        sp.state = n_;
+        sp.vdim = vdim_;
+        sp.x_off = 0;
+        sp.b_off = inner_;
+        sp.c_off = inner_ + gn_;
+        sp.s_off = (int64_t)(taps_ - 1) * (inner_ + 2 * gn_);
+        Tensor y = ops.ssd_scan(xbc, dt, head_vector(0), head_vector(1), head_vector(2), sp, view, ctx);
+        Tensor g = ops.gate_group_norm(y, columns(in, 0, inner_), tensor("norm"), norm_groups_, eps_, x.dtype);
+        if (residual.defined()) return PartOut(ops.linear_residual(Rows(g), tensor("o"), nullptr, residual, out_scale));
+        Tensor out = ops.linear(Rows(g), tensor("o"), nullptr, nullptr, (int)DType::F32);        // the block sums itself
+        if (out_scale != 1.0f) ops.scale_rows(out, out_scale);
+        return PartOut(out);
+    }
+
+private:
+    int heads_, vdim_, n_, groups_, taps_, norm_groups_;
+    int64_t inner_, gn_;
+    float eps_;
+};
+
 // ------------------------------------------------------------------ mixers side by side
 // out = residual + sum_i scale_i * member_i(h).  Members are named by the specification's "members" (roles of sub-parts,
 // in order) and weighted by "scales"; each keeps the part of the cache entry that it asked for (a member that asks for
@@ -341,8 +420,11 @@ public:
         // g sigmoid(a g) (u + 1), g = min(gate, L), u = clamp(up, -L, L) ("shared_limit": the L of the expert that every row
         // uses).  "shared_gate" names a row [1, width] whose sigmoid multiplies that expert's result.
         const std::string score = s.params.get_string("score", "softmax");
-        if (score != "softmax" && score != "sigmoid" && score != "softmax_biased")
-            throw ConfigError("routed_experts: 'score' is \"softmax\", \"sigmoid\" or \"softmax_biased\"");
+        // "score": "table": no router; the integer tensor "table" [vocab, top] ("vocab") gives every token id its experts, each with the
+        // weight 1 / top, so a step whose token ids the host knows needs no look at the device to group its rows.
+        if (score != "softmax" && score != "sigmoid" && score != "softmax_biased" && score != "table")
+            throw ConfigError("routed_experts: 'score' is \"softmax\", \"sigmoid\", \"softmax_biased\" or \"table\"");
+        tabled_ = score == "table";
         sigmoid_ = score == "sigmoid";
         biased_ = score == "softmax_biased";
         identity_ = (int)s.params.get_int("identity", 0);
@@ -368,7 +450,11 @@ public:
             throw ConfigError("routed_experts: groups, a choice bias and a weight multiplier belong to sigmoid scores");
         if (!shared_gate_.empty() && (shared_inner_ <= 0 || router_bias_)) throw ConfigError("routed_experts: 'shared_gate' belongs to an expert that every row uses and a router without bias");
         const int64_t w = e.width, outputs = (int64_t)experts_ + identity_;
-        if (shared_gate_.empty()) {
+        if (tabled_) {
+            const int64_t vocab = s.params.get_int("vocab", 0);
+            if (vocab <= 0 || router_bias_ || !choice_bias_.empty() || !shared_gate_.empty()) throw ConfigError("routed_experts: a table of token ids needs 'vocab', and has no router's bias and no gate");
+            declare("table", {vocab, (int64_t)top_}, true).below = experts_;
+        } else if (shared_gate_.empty()) {
             declare("router", {outputs, w});
         } else {                                                 // the gate is one more row of the router's product
             declare_stacked("w_router", outputs + 1, w);
@@ -394,7 +480,8 @@ public:
     }
     PartOut forward(Ops& ops, const Rows& h, const Tensor& residual_in, const StepContext& ctx, Norm*) override {
         Tensor x = ops.materialize(h);
-        Tensor logits = ops.linear(Rows(x), tensor(shared_gate_.empty() ? "router" : "w_router"), router_bias_ ? &tensor("router.b") : nullptr, nullptr, (int)DType::F32);
+        Tensor logits;
+        if (!tabled_) logits = ops.linear(Rows(x), tensor(shared_gate_.empty() ? "router" : "w_router"), router_bias_ ? &tensor("router.b") : nullptr, nullptr, (int)DType::F32);
         // what the chosen experts' results are added to: the stream; with an expert that every row uses, its result on top
         // of the stream; without a stream (a block that sums itself), that result alone or zeros, 32-bit
         Tensor residual = residual_in;
@@ -417,14 +504,16 @@ public:
         // needs the host, so a one-token step (which may be captured in a graph) never groups.
         const double per_row = 3.0 * (double)inner_ * (double)x.cols();
         const double dense_work = (double)x.rows() * experts_ * per_row;
-        const double grouped_work = (double)x.rows() * top_ * per_row + (2.0 * experts_ * 25e9 + 100e9) / 2.0;
+        const std::vector<int> counts = choices_per_expert(ctx);          // empty: only the device knows
+        const double grouped_work = (double)x.rows() * top_ * per_row + (2.0 * experts_ * 25e9 + (counts.empty() ? 100e9 : 0.0)) / 2.0;
         // FRIDAY_EXPERTS=grouped|dense|pairs forces a form where it can run (for comparisons and tests)
         const char* force = getenv("FRIDAY_EXPERTS");
         const std::string forced = force ? force : "";
         const bool may_group = tensor_cores && !ctx.decode && ctx.rows == (int)x.rows() && ctx.n_seqs > 0;
         const bool grouped = may_group && (forced == "grouped" || (forced.empty() && grouped_work < dense_work));
         const bool dense = tensor_cores && !grouped && (forced == "dense" || (forced.empty() && experts_ <= 16 * top_));
-        Ops::Routing r = sigmoid_ ? ops.route_scored(logits, top_, choice_bias_.empty() ? nullptr : &tensor(choice_bias_), groups_, keep_,
+        Ops::Routing r = tabled_ ? ops.route_table(ctx.tokens, x.rows(), tensor("table"), experts_, dense)
+                        : sigmoid_ ? ops.route_scored(logits, top_, choice_bias_.empty() ? nullptr : &tensor(choice_bias_), groups_, keep_,
                                                      weight_scale_, dense)
                         : biased_ ? ops.route_biased(logits, experts_, identity_, top_, choice_bias_.empty() ? nullptr : &tensor(choice_bias_), dense)
                                   : ops.route(logits, top_, softmax_all_, dense);
@@ -448,7 +537,7 @@ public:
             residual = with_shared(residual_in);
         }
         if (grouped)
-            return PartOut(ops.experts_grouped(x, r, tensor("w_gate_up"), tensor("w_down"), residual, top_, inner_, act_, limit_, slope_));
+            return PartOut(ops.experts_grouped(x, r, tensor("w_gate_up"), tensor("w_down"), residual, top_, inner_, act_, limit_, slope_, counts.empty() ? nullptr : &counts));
         if (dense) {
             Tensor act = ops.linear_swiglu(Rows(x), tensor("w_gate_up"), act_, limit_, slope_);
             ops.scale_by_route(act, r.dense, experts_, inner_);
@@ -458,9 +547,30 @@ public:
         return PartOut(ops.expert_down_combine(act, r, tensor("w_down"), residual, top_, inner_));
     }
 
+    void finalize(Ops& ops) override {
+        FeedForward::finalize(ops);
+        if (!tabled_) return;
+        const Tensor& t = tensor("table");
+        table_.resize((size_t)t.numel());
+        cuda_check(cudaMemcpyAsync(table_.data(), t.data, table_.size() * sizeof(int), cudaMemcpyDeviceToHost, ops.stream()), "cudaMemcpyAsync");
+        cuda_check(cudaStreamSynchronize(ops.stream()), "cudaStreamSynchronize");
+        for (int id : table_)
+            if (id < 0 || id >= experts_) throw WeightsError(format("%stable: expert %d of %d", prefix.c_str(), id, experts_));
+    }
+
 private:
+    // how often the step's tokens choose each expert, where a table and the host's token ids tell
+    std::vector<int> choices_per_expert(const StepContext& ctx) const {
+        if (!tabled_ || (int)ctx.host_tokens.size() != ctx.rows || ctx.decode) return {};
+        std::vector<int> n((size_t)experts_, 0);
+        for (int token : ctx.host_tokens)
+            for (int j = 0; j < top_; ++j) ++n[(size_t)table_[(size_t)token * top_ + j]];
+        return n;
+    }
+
     int experts_, top_, inner_;
-    bool softmax_all_;
+    bool softmax_all_, tabled_ = false;
+    std::vector<int> table_;
     bool sigmoid_ = false, router_bias_ = true, biased_ = false;
     int identity_ = 0, act_ = 1;
     float limit_ = 0.f, shared_limit_ = 0.f, slope_ = 1.f;
@@ -508,6 +618,7 @@ private:
 namespace {
 PartRegistrar s1("mixer", "gated_linear_attention", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new GatedLinearAttention(s, e); });
 PartRegistrar s1b("mixer", "decayed_linear_attention", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new DecayedLinearAttention(s, e); });
+PartRegistrar s1c("mixer", "state_space_dual", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new StateSpaceDual(s, e); });
 PartRegistrar s2("mixer", "shift_decay_mix", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new ShiftDecayMix(s, e); });
 PartRegistrar s3("mixer", "parallel", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new ParallelMixer(s, e); });
 PartRegistrar s4("feed_forward", "routed_experts", [](const PartSpec& s, const BuildEnv& e) -> Part* { return new RoutedExperts(s, e); });

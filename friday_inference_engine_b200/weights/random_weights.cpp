@@ -43,6 +43,18 @@ void random_tensor_host(uint64_t seed, const std::string& name, bool one, int64_
 
 namespace {
 
+// ids 0 .. below - 1, those of a row all different (consecutive from a random one on) while the range has as many
+std::vector<int32_t> random_ids(uint64_t seed, const std::string& name, int64_t rows, int64_t cols, int64_t below) {
+    const uint64_t key = random_stream_key(seed, name);
+    std::vector<int32_t> out((size_t)(rows * cols));
+    for (int64_t r = 0; r < rows; ++r) {
+        uint32_t c[4] = {(uint32_t)r, (uint32_t)((uint64_t)r >> 32), 0u, 0u};
+        fr_philox4x32_10(c, (uint32_t)key, (uint32_t)(key >> 32));
+        for (int64_t j = 0; j < cols; ++j) out[(size_t)(r * cols + j)] = (int32_t)(((int64_t)(c[0] >> 1) + j) % below);
+    }
+    return out;
+}
+
 class RandomSource : public WeightSource {
 public:
     RandomSource(const std::vector<Part::Named>& expected, uint64_t seed, const std::string& dtype, bool on_device)
@@ -74,6 +86,13 @@ public:
         if (n == 0) return;
         const int64_t cols = t.shape.size() >= 2 ? t.shape.back() : 1, rows = n / cols;
         const size_t es = dtype_size(dst.dtype);
+        if (d.integer && d.below > 0) {
+            const std::vector<int32_t> v = random_ids(seed_, name, rows, cols, d.below);
+            cuda_check(cudaMemcpy2DAsync(dst.data, (size_t)dst.ld * es, v.data(), (size_t)cols * es, (size_t)cols * es, (size_t)rows,
+                                         cudaMemcpyHostToDevice, stream), "cudaMemcpy2DAsync");
+            cuda_check(cudaStreamSynchronize(stream), "cudaStreamSynchronize");
+            return;
+        }
         if (d.integer) {
             cuda_check(cudaMemset2DAsync(dst.data, (size_t)dst.ld * es, 0, (size_t)cols * es, (size_t)rows, stream), "cudaMemset2DAsync");
             return;
@@ -160,6 +179,11 @@ void write_random_model(const std::string& dir, const Json& config_json, uint64_
         if (e.decl.integer) {
             t.dtype = "I32";
             t.bytes.assign((size_t)n * 4, 0);
+            if (e.decl.below > 0 && n > 0) {
+                const int64_t cols = t.shape.size() >= 2 ? t.shape.back() : 1;
+                const std::vector<int32_t> v = random_ids(seed, e.name, n / cols, cols, e.decl.below);
+                memcpy(t.bytes.data(), v.data(), t.bytes.size());
+            }
         } else {
             std::vector<float> f((size_t)n);
             random_tensor_host(seed, e.name, e.decl.one, n, f.data());
