@@ -755,6 +755,60 @@ def zudovik_numbers(cfg, batch, context, prompt_len):
     return {"step_bytes": weight_bytes + state_bytes + kv_bytes, "flops_per_token": flops}
 
 
+def dapozen_config(width, layers=7, vocab=32768, experts=8, top=2):
+    """A Dapozen configuration whose layers have sizes like a real model's of this width: attention within runs of 2,048 positions
+    (heads of 128 on a quarter as many key/value heads, half of a head rotated, convolutions of 4 taps) and, as every third layer from the
+    second on, state space duality with twice the width in heads of 64 and a state of 128 rows in two groups; a dense gated feed-forward of
+    three times the width in the even layers and, in the odd ones, `experts` experts of inner size width, `top` of them per token id, with
+    one that every token uses."""
+    heads, kv = max(1, width // 128), max(1, width // 512)
+    att = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "conv": 4, "scale": 128 ** -0.5, "rot": {"base": 10000.0, "dims": 64},
+           "mask": {"size": 2048}}
+    ssd = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 2, "norm_groups": 2, "conv": 4}
+    dense = {"kind": "dense", "ff": 3 * width}
+    moe = {"kind": "moe", "expert": {"ff": width, "limit": 7.0}, "router": {"experts": experts, "top": top}, "shared": {"ff": width, "limit": 7.0}}
+    ls = [{"type": "mamba2" if i % 3 == 1 else "attention", "mixer": ssd if i % 3 == 1 else att, "mlp": dense if i % 2 == 0 else moe} for i in range(layers)]
+    return {"architecture": "Dapozen", "vocab": vocab, "width": width, "embedding": {"scale": 12.0}, "norm": {"eps": 1e-6}, "layers": ls,
+            "logit_softcap": 25.0}
+
+
+def dapozen_numbers(cfg, batch, context, prompt_len):
+    """What a decode step of `batch` sequences must read (weights, the experts that the batch touches, cached keys and values in sight, the
+    states) and what a prompt token costs (the attention's share for a prompt of prompt_len tokens; the experts of the token's id only)."""
+    w, v = cfg["width"], cfg["vocab"]
+    weight_bytes = 2 * v * w
+    flops = 2 * v * w
+    state_bytes = kv_bytes = 0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        H, vd = m["heads"], m["vdim"]
+        if L["type"] == "mamba2":
+            inner, gn, n = H * vd, m["groups"] * m["state"], m["state"]
+            mat = (2 * inner + 2 * gn + H) * w + w * inner
+            state_bytes += batch * 4 * 2 * (H * n * vd + (m["conv"] - 1) * (inner + 2 * gn))
+            mix = 4 * H * n * vd
+        else:
+            G, d = m["kv_heads"], m["dim"]
+            mat = (H * d + G * (d + vd) + H * vd) * w + w * H * vd
+            size = m["mask"]["size"]
+            seen = (context - 1) % size + 1
+            kv_bytes += batch * seen * G * (d + vd) * 2
+            state_bytes += batch * 4 * 2 * (m["conv"] - 1) * (H * d + G * (d + vd))
+            mix = 2 * H * (d + vd) * min(prompt_len, size) // 2
+        ff = ff_read = 0
+        mlp = L.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            ff = ff_read = 3 * mlp["ff"] * w
+        elif mlp:
+            r, f = mlp["router"], 3 * mlp["expert"]["ff"] * w
+            base = 3 * mlp["shared"]["ff"] * w if mlp.get("shared") else 0
+            ff = base + r["top"] * f
+            ff_read = base + r["experts"] * (1.0 - (1.0 - r["top"] / r["experts"]) ** batch) * f
+        weight_bytes += 2 * (mat + ff_read)
+        flops += 2 * (mat + ff) + mix
+    return {"step_bytes": weight_bytes + state_bytes + kv_bytes, "flops_per_token": flops}
+
+
 def tikunex_numbers(cfg, batch, context):
     """What a decode step of `batch` sequences must read and what a prompt token costs, per run of the layers."""
     w, v = cfg["width"], cfg["vocab"]
@@ -800,7 +854,7 @@ def tikunex_numbers(cfg, batch, context):
 
 
 def design_compare(Engine, args):
-    """Zudovik, Vulanex, Ditenex, Beletar and Tikunex beside the Qwen2.5 dense decoder at equal width and depth (random weights): one prompt and decode
+    """Dapozen, Zudovik, Vulanex, Ditenex, Beletar and Tikunex beside the Qwen2.5 dense decoder at equal width and depth (random weights): one prompt and decode
     steps, with the share of each kind of kernel in the prompt (event-bracketed).  One line of text per measurement.
     --designs picks among them."""
     pk = peaks()
@@ -808,6 +862,7 @@ def design_compare(Engine, args):
     for width in [int(v) for v in args.design_compare.split(",") if v]:
         layers = args.layers or 4
         designs = [
+            ("dapozen", dapozen_config(width, 2 * layers - 1)),
             ("zudovik", zudovik_config(width, 2 * layers - 1)),
             ("vulanex", vulanex_config(width, 2 * layers - 1)),
             ("ditenex", ditenex_config(width, 2 * layers - 1)),
@@ -820,7 +875,10 @@ def design_compare(Engine, args):
             if name not in args.designs.split(","):
                 continue
             eng = Engine(config=cfg, seed=0, dtype="bfloat16", max_ctx=4096, max_batch=batch, max_tokens=batch * 4096 + 8192)
-            if name == "zudovik":
+            if name == "dapozen":
+                nums = dapozen_numbers(cfg, batch, context + 64, prompt_len)
+                flops_tok, step_bytes = nums["flops_per_token"], nums["step_bytes"]
+            elif name == "zudovik":
                 nums = zudovik_numbers(cfg, batch, context + 64, prompt_len)
                 flops_tok, step_bytes = nums["flops_per_token"], nums["step_bytes"]
             elif name == "vulanex":
@@ -898,7 +956,7 @@ def main():
     ap.add_argument("--design-compare", default="", dest="design_compare",
                     help="widths, e.g. 1024,2048,4096: a Zudovik, a Vulanex, a Ditenex, a Beletar and a Tikunex model with layers of that size beside the Qwen2.5 "
                          "decoder of equal width (prompt, decode steps, kernel shares): lines of text")
-    ap.add_argument("--designs", default="zudovik,vulanex,ditenex,beletar,tikunex,qwen2", help="which designs --design-compare runs")
+    ap.add_argument("--designs", default="dapozen,zudovik,vulanex,ditenex,beletar,tikunex,qwen2", help="which designs --design-compare runs")
     ap.add_argument("--timeline", action="store_true",
                     help="print the kernels of one decode step as they run inside the captured graph (torch profiler)")
     args = ap.parse_args()

@@ -324,6 +324,254 @@ int launch_rows(const ConvArgs& p, cudaStream_t stream) {
     return FR_OK;
 }
 
+// ------------------------------------------------------------------ eight channels per thread
+// The usual shapes (up to four taps, rows in whole 16-byte pieces; heads of a power of two): a thread owns eight channels of a run of
+// rows, asks for all of its rows at once and keeps the last three inputs in registers, so an input is read, and widened, once for all
+// its taps.
+template <typename T> struct Eight;
+template <> struct Eight<float> { float4 a, b; };
+template <> struct Eight<bf16> { uint4 a; };
+__device__ __forceinline__ void load_eight(const float* p, Eight<float>& v) { v.a = *(const float4*)p; v.b = *(const float4*)(p + 4); }
+__device__ __forceinline__ void load_eight(const bf16* p, Eight<bf16>& v) { v.a = *(const uint4*)p; }
+__device__ __forceinline__ void widen(const Eight<float>& v, float (&f)[8]) {
+    f[0] = v.a.x; f[1] = v.a.y; f[2] = v.a.z; f[3] = v.a.w; f[4] = v.b.x; f[5] = v.b.y; f[6] = v.b.z; f[7] = v.b.w;
+}
+__device__ __forceinline__ void widen(const Eight<bf16>& v, float (&f)[8]) {
+    const uint32_t w[4] = {v.a.x, v.a.y, v.a.z, v.a.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        f[2 * i] = __uint_as_float(w[i] << 16);
+        f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void store_eight(float* p, const float (&f)[8]) {
+    *(float4*)p = make_float4(f[0], f[1], f[2], f[3]);
+    *(float4*)(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+}
+__device__ __forceinline__ void store_eight(bf16* p, const float (&f)[8]) {
+    uint4 r;
+    pack(f[0], f[1], r.x);
+    pack(f[2], f[3], r.y);
+    pack(f[4], f[5], r.z);
+    pack(f[6], f[7], r.w);
+    *(uint4*)p = r;
+}
+
+// What a row means to the kernels below; read ahead of the wait for the kernel before (the step's geometry is final by then)
+struct RowPlace {
+    int seq, known, pos, slot;
+};
+__device__ __forceinline__ RowPlace place_of(const ConvArgs& p, int row) {
+    RowPlace r;
+    r.seq = p.row_seq[row];
+    r.known = r.seq >= 0 ? row - p.seq_start[r.seq] : 0;
+    r.pos = p.row_pos != nullptr ? p.row_pos[row] : 0;
+    r.slot = r.seq >= 0 ? p.seq_slots[r.seq] : 0;
+    return r;
+}
+
+template <typename T>
+struct Walk {
+    float w[4][8];                   // taps, the last one the present row's; missing ones count zero
+    float back[3][8];                // the inputs three, two and one row before the present one
+    __device__ __forceinline__ void load_taps(const ConvArgs& p, int c) {
+        if (p.taps == 4) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                float v[4];
+                p.taps_w.four((c + i) * 4, v);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) w[j][i] = v[j];
+            }
+            return;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) w[j][i] = j >= 4 - p.taps ? p.taps_w.at((c + i) * p.taps + j - (4 - p.taps)) : 0.f;
+    }
+    // the inputs before `row`: rows of this step as far as its sequence has them, then the sequence's history
+    __device__ __forceinline__ void begin(const ConvArgs& p, const T* x, int row, int known, const float* hist, int c) {
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            const int b = 3 - k;
+            if (b <= known) {
+                Eight<T> v;
+                load_eight(x + (size_t)(row - b) * p.ld + p.off + c, v);
+                widen(v, back[k]);
+            } else if (b <= p.taps - 1 + known && b < p.taps) {
+                Eight<float> v;
+                load_eight(hist + (size_t)(p.taps - 1 + known - b) * p.channels + c, v);
+                widen(v, back[k]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) back[k][i] = 0.f;
+            }
+        }
+    }
+    // the convolution at a row whose input is `u`
+    __device__ __forceinline__ void step(const float (&u)[8], float (&y)[8]) const {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = fmaf(w[3][i], u[i], fmaf(w[2][i], back[2][i], fmaf(w[1][i], back[1][i], w[0][i] * back[0][i])));
+    }
+    __device__ __forceinline__ void take(const float (&u)[8]) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            back[0][i] = back[1][i];
+            back[1][i] = back[2][i];
+            back[2][i] = u[i];
+        }
+    }
+    // after take(): the last taps - 1 inputs are the sequence's history
+    __device__ __forceinline__ void leave(const ConvArgs& p, float* hist, int c) const {
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            const int j = k - (3 - (p.taps - 1));
+            if (j >= 0) store_eight(hist + (size_t)j * p.channels + c, back[k]);
+        }
+    }
+};
+
+constexpr int VEC_THREADS = 128;
+
+// LANES: threads of a head (its channels / 8)
+template <typename T, int LANES, int R>
+__global__ void __launch_bounds__(VEC_THREADS) conv_heads_vec_kernel(ConvArgs p) {
+    __shared__ float2 turn[R][128];          // cosine and sine of every row's angles
+    const int row0 = blockIdx.x * R, n = min(R, p.rows - row0);
+    const int c = 8 * (blockIdx.y * VEC_THREADS + threadIdx.x);
+    const int half = p.freq != nullptr ? p.rot / 2 : 0, nq = p.heads * p.dim, nk = p.kv_heads * p.dim, nv = p.kv_heads * p.vdim;
+    const bool live = c < nq + nk + nv, is_q = c < nq, is_v = c >= nq + nk;
+    Walk<T> walk;
+    RowPlace first = place_of(p, row0);
+    if (live) walk.load_taps(p, c);
+    if (half > 0 && 8 * (int)blockIdx.y * VEC_THREADS < nq + nk) {
+        for (int idx = threadIdx.x; idx < n * half; idx += VEC_THREADS) {
+            const int r = idx / half, i = idx - r * half;
+            float s, co;
+            sincosf((float)p.row_pos[row0 + r] * p.freq[i], &s, &co);
+            turn[r][i] = make_float2(co, s);
+        }
+    }
+    fr_pdl_wait();
+    fr_pdl_launch();
+    __syncthreads();
+    if (!live) return;                       // whole heads: a head's lanes are all live or none
+    const T* x = (const T*)p.x;
+    Eight<T> raw[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+        if (r < n) load_eight(x + (size_t)(row0 + r) * p.ld + p.off + c, raw[r]);
+    const int d = is_v ? 0 : c % p.dim;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+        if (r >= n) break;
+        const int row = row0 + r;
+        const RowPlace at = r == 0 ? first : place_of(p, row);
+        if (at.seq < 0) continue;            // (a dead row: the walk begins anew at the next sequence's first row)
+        float* hist = p.state + (size_t)at.slot * p.state_stride + p.hist_off;
+        if (r == 0 || at.known == 0) walk.begin(p, x, row, at.known, hist, c);
+        float u[8], y[8];
+        widen(raw[r], u);
+        walk.step(u, y);
+        walk.take(u);
+        if (p.shift) walk.leave(p, hist, c);
+        if (!is_v) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (d / 2 + i < half) {
+                    const float2 t = turn[r][d / 2 + i];
+                    const float a = y[2 * i], b = y[2 * i + 1];
+                    fr_rotate(a, b, t.x, t.y, y[2 * i], y[2 * i + 1]);
+                }
+            }
+            if (p.norm) {
+                float ss = 0.f;
+#pragma unroll
+                for (int i = 0; i < 8; ++i) ss = fmaf(y[i], y[i], ss);
+                const unsigned lanes = LANES == 32 ? 0xffffffffu : ((1u << LANES) - 1u) << ((threadIdx.x & 31) / LANES * LANES);
+#pragma unroll
+                for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(lanes, ss, o);
+                const float inv = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) y[i] *= inv;
+            }
+        }
+        if (is_q) {
+            store_eight((T*)p.q_out + (size_t)row * nq + c, y);
+        } else {
+            const size_t to = (size_t)p.block_table[(size_t)at.seq * p.table_width + at.pos / PAGE_ROWS] * PAGE_ROWS + at.pos % PAGE_ROWS;
+            if (is_v) store_eight((T*)p.v_pool + to * nv + (c - nq - nk), y);
+            else store_eight((T*)p.k_pool + to * nk + (c - nq), y);
+        }
+    }
+}
+
+template <typename T, int LANES>
+int launch_heads_vec(const ConvArgs& p, cudaStream_t stream) {
+    const int blocks = (p.channels / 8 + VEC_THREADS - 1) / VEC_THREADS;
+    const bool single = p.shift || (long long)p.rows * blocks < (long long)fr_sm_count() * 8;
+    if (single) FR_CUDA(fr_launch(conv_heads_vec_kernel<T, LANES, 1>, dim3(p.rows, blocks), dim3(VEC_THREADS), 0, stream, p));
+    else FR_CUDA(fr_launch(conv_heads_vec_kernel<T, LANES, 8>, dim3((p.rows + 7) / 8, blocks), dim3(VEC_THREADS), 0, stream, p));
+    FR_CHECK_LAUNCH("short_conv heads");
+    return FR_OK;
+}
+
+// silu: exact for 32-bit rows; for rows about to be rounded to bf16 with the hardware's exponential and reciprocal
+template <typename T> __device__ __forceinline__ float silu_to(float z);
+template <> __device__ __forceinline__ float silu_to<float>(float z) { return z / (1.0f + expf(-z)); }
+template <> __device__ __forceinline__ float silu_to<bf16>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
+template <typename TI, typename TO, int R>
+__global__ void __launch_bounds__(VEC_THREADS) conv_rows_vec_kernel(ConvArgs p) {
+    const int row0 = blockIdx.x * R, n = min(R, p.rows - row0);
+    const int c = 8 * (blockIdx.y * VEC_THREADS + threadIdx.x);
+    const bool live = c < p.channels;
+    Walk<TI> walk;
+    const RowPlace first = place_of(p, row0);
+    float bias[8];
+    if (live) {
+        walk.load_taps(p, c);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) bias[i] = p.bias.p != nullptr ? p.bias.at(c + i) : 0.f;
+    }
+    fr_pdl_wait();
+    fr_pdl_launch();
+    if (!live) return;
+    const TI* x = (const TI*)p.x;
+    Eight<TI> raw[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+        if (r < n) load_eight(x + (size_t)(row0 + r) * p.ld + p.off + c, raw[r]);
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+        if (r >= n) break;
+        const int row = row0 + r;
+        const RowPlace at = r == 0 ? first : place_of(p, row);
+        if (at.seq < 0) continue;
+        float* hist = p.state + (size_t)at.slot * p.state_stride + p.hist_off;
+        if (r == 0 || at.known == 0) walk.begin(p, x, row, at.known, hist, c);
+        float u[8], y[8];
+        widen(raw[r], u);
+        walk.step(u, y);
+        walk.take(u);
+        if (p.shift) walk.leave(p, hist, c);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = silu_to<TO>(y[i] + bias[i]);
+        store_eight((TO*)p.out + (size_t)row * p.channels + c, y);
+    }
+}
+
+template <typename TI, typename TO>
+int launch_rows_vec(const ConvArgs& p, cudaStream_t stream) {
+    const int blocks = (p.channels / 8 + VEC_THREADS - 1) / VEC_THREADS;
+    const bool single = p.shift || (long long)p.rows * blocks < (long long)fr_sm_count() * 8;
+    if (single) FR_CUDA(fr_launch(conv_rows_vec_kernel<TI, TO, 1>, dim3(p.rows, blocks), dim3(VEC_THREADS), 0, stream, p));
+    else FR_CUDA(fr_launch(conv_rows_vec_kernel<TI, TO, 8>, dim3((p.rows + 7) / 8, blocks), dim3(VEC_THREADS), 0, stream, p));
+    FR_CHECK_LAUNCH("short_conv rows");
+    return FR_OK;
+}
+
 // ------------------------------------------------------------------ history
 template <typename T>
 __global__ void __launch_bounds__(256) conv_history_kernel(ConvArgs p) {
@@ -385,6 +633,16 @@ FR_EXPORT int short_conv_heads(const void* x, int ld, int off, const void* taps_
     p.pairs = ((ld | off | dim | vdim) & 1) == 0 && (at & 7) == 0;
     const int big = dim > vdim ? dim : vdim;
     int done;
+    const bool eights = taps <= 4 && ((ld | off | vdim) & 7) == 0 && ((at | (uintptr_t)state) & 15) == 0 && ((state_stride | hist_off | p.channels) & 3) == 0 &&
+                        (rot <= 256 || freq == nullptr);
+    if (eights && (dim == 32 || dim == 64 || dim == 128 || dim == 256) && (dtype == FR_F32 || dtype == FR_BF16)) {
+        const bool wide = dtype == FR_F32;
+        if (dim == 32) done = wide ? launch_heads_vec<float, 4>(p, stream) : launch_heads_vec<bf16, 4>(p, stream);
+        else if (dim == 64) done = wide ? launch_heads_vec<float, 8>(p, stream) : launch_heads_vec<bf16, 8>(p, stream);
+        else if (dim == 128) done = wide ? launch_heads_vec<float, 16>(p, stream) : launch_heads_vec<bf16, 16>(p, stream);
+        else done = wide ? launch_heads_vec<float, 32>(p, stream) : launch_heads_vec<bf16, 32>(p, stream);
+        return done != FR_OK ? done : history(p, n_seqs, dtype, stream);
+    }
     if (dtype == FR_F32) done = big <= 64 ? launch_heads<float, 1>(p, stream) : big <= 128 ? launch_heads<float, 2>(p, stream) : launch_heads<float, 4>(p, stream);
     else if (dtype == FR_BF16) done = big <= 64 ? launch_heads<bf16, 1>(p, stream) : big <= 128 ? launch_heads<bf16, 2>(p, stream) : launch_heads<bf16, 4>(p, stream);
     else FR_REFUSE("short_conv: unknown dtype %d", dtype);
@@ -406,6 +664,13 @@ FR_EXPORT int short_conv_rows(const void* x, int ld, int off, int channels, cons
     if (channels > 65535 * ROW_THREADS) FR_REFUSE("short_conv: %d channels", channels);
     p.pairs = ((ld | off | channels) & 1) == 0 && (((uintptr_t)x | (uintptr_t)out) & 7) == 0;
     int done;
+    if (taps <= 4 && ((ld | off | channels) & 7) == 0 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)state) & 15) == 0 && ((state_stride | hist_off) & 3) == 0) {
+        if (in_dtype == FR_F32 && out_dtype == FR_F32) done = launch_rows_vec<float, float>(p, stream);
+        else if (in_dtype == FR_F32 && out_dtype == FR_BF16) done = launch_rows_vec<float, bf16>(p, stream);
+        else if (in_dtype == FR_BF16 && out_dtype == FR_BF16) done = launch_rows_vec<bf16, bf16>(p, stream);
+        else FR_REFUSE("short_conv: rows of dtype %d from inputs of dtype %d", out_dtype, in_dtype);
+        return done != FR_OK ? done : history(p, n_seqs, in_dtype, stream);
+    }
     if (in_dtype == FR_F32 && out_dtype == FR_F32) done = launch_rows<float, float>(p, stream);
     else if (in_dtype == FR_F32 && out_dtype == FR_BF16) done = launch_rows<float, bf16>(p, stream);
     else if (in_dtype == FR_BF16 && out_dtype == FR_BF16) done = launch_rows<bf16, bf16>(p, stream);

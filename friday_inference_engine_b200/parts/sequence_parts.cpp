@@ -501,11 +501,13 @@ public:
         // every row, or the chosen ones plus what two launches per expert and the host's wait cost (measured on a B200:
         // grouping broke even at width 2,048 with 8 experts of inner size 2,048, 2 chosen, 2,048 rows, and won a fifth
         // of the prompt's time at width 4,096; a launch counts as 25 G multiply-adds, the wait as 100 G).  Grouping
-        // needs the host, so a one-token step (which may be captured in a graph) never groups.
+        // needs the host, so a one-token step (which may be captured in a graph) never groups.  Where the host knows the counts
+        // without looking (a table of token ids) there is no wait and the queue stays full: a launch counts as 17 G (the two forms
+        // were within a fiftieth of each other at width 2,048, 3.56 and 3.63 ms a prompt).
         const double per_row = 3.0 * (double)inner_ * (double)x.cols();
         const double dense_work = (double)x.rows() * experts_ * per_row;
         const std::vector<int> counts = choices_per_expert(ctx);          // empty: only the device knows
-        const double grouped_work = (double)x.rows() * top_ * per_row + (2.0 * experts_ * 25e9 + (counts.empty() ? 100e9 : 0.0)) / 2.0;
+        const double grouped_work = (double)x.rows() * top_ * per_row + (counts.empty() ? 2.0 * experts_ * 25e9 + 100e9 : 2.0 * experts_ * 17e9) / 2.0;
         // FRIDAY_EXPERTS=grouped|dense|pairs forces a form where it can run (for comparisons and tests)
         const char* force = getenv("FRIDAY_EXPERTS");
         const std::string forced = force ? force : "";
