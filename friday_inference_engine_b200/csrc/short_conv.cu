@@ -357,18 +357,29 @@ __device__ __forceinline__ void store_eight(bf16* p, const float (&f)[8]) {
     *(uint4*)p = r;
 }
 
-// What a row means to the kernels below; read ahead of the wait for the kernel before (the step's geometry is final by then)
+// What a row means to the kernels below: rows of its sequence before it in this step (-1: a dead row), its slot, and where its key and
+// value lie in the cache.  A block makes it once for each of its rows, ahead of the wait for the kernel before (the step's geometry is
+// final by then).
 struct RowPlace {
-    int seq, known, pos, slot;
+    int known, slot, to;
 };
 __device__ __forceinline__ RowPlace place_of(const ConvArgs& p, int row) {
     RowPlace r;
-    r.seq = p.row_seq[row];
-    r.known = r.seq >= 0 ? row - p.seq_start[r.seq] : 0;
-    r.pos = p.row_pos != nullptr ? p.row_pos[row] : 0;
-    r.slot = r.seq >= 0 ? p.seq_slots[r.seq] : 0;
+    const int seq = p.row_seq[row];
+    r.known = seq >= 0 ? row - p.seq_start[seq] : -1;
+    r.slot = seq >= 0 ? p.seq_slots[seq] : 0;
+    r.to = 0;
+    if (seq >= 0 && p.block_table != nullptr) {
+        const int pos = p.row_pos[row];
+        r.to = p.block_table[(size_t)seq * p.table_width + pos / PAGE_ROWS] * PAGE_ROWS + pos % PAGE_ROWS;
+    }
     return r;
 }
+// 1 / sqrt(mean square + eps): exact for 32-bit rows, the hardware's reciprocal square root (its error is far below the rounding that
+// follows) for rows in bf16
+template <typename T> __device__ __forceinline__ float inverse_rms(float mean_square_eps);
+template <> __device__ __forceinline__ float inverse_rms<float>(float v) { return 1.0f / sqrtf(v); }
+template <> __device__ __forceinline__ float inverse_rms<bf16>(float v) { return rsqrtf(v); }
 
 template <typename T>
 struct Walk {
@@ -438,12 +449,13 @@ constexpr int VEC_THREADS = 128;
 template <typename T, int LANES, int R>
 __global__ void __launch_bounds__(VEC_THREADS) conv_heads_vec_kernel(ConvArgs p) {
     __shared__ float2 turn[R][128];          // cosine and sine of every row's angles
+    __shared__ RowPlace place[R];
     const int row0 = blockIdx.x * R, n = min(R, p.rows - row0);
     const int c = 8 * (blockIdx.y * VEC_THREADS + threadIdx.x);
     const int half = p.freq != nullptr ? p.rot / 2 : 0, nq = p.heads * p.dim, nk = p.kv_heads * p.dim, nv = p.kv_heads * p.vdim;
     const bool live = c < nq + nk + nv, is_q = c < nq, is_v = c >= nq + nk;
     Walk<T> walk;
-    RowPlace first = place_of(p, row0);
+    if ((int)threadIdx.x < n) place[threadIdx.x] = place_of(p, row0 + threadIdx.x);
     if (live) walk.load_taps(p, c);
     if (half > 0 && 8 * (int)blockIdx.y * VEC_THREADS < nq + nk) {
         for (int idx = threadIdx.x; idx < n * half; idx += VEC_THREADS) {
@@ -463,12 +475,13 @@ __global__ void __launch_bounds__(VEC_THREADS) conv_heads_vec_kernel(ConvArgs p)
     for (int r = 0; r < R; ++r)
         if (r < n) load_eight(x + (size_t)(row0 + r) * p.ld + p.off + c, raw[r]);
     const int d = is_v ? 0 : c % p.dim;
+    const float inv_dim = 1.0f / (float)p.dim;
 #pragma unroll
     for (int r = 0; r < R; ++r) {
         if (r >= n) break;
         const int row = row0 + r;
-        const RowPlace at = r == 0 ? first : place_of(p, row);
-        if (at.seq < 0) continue;            // (a dead row: the walk begins anew at the next sequence's first row)
+        const RowPlace at = place[r];
+        if (at.known < 0) continue;          // (a dead row: the walk begins anew at the next sequence's first row)
         float* hist = p.state + (size_t)at.slot * p.state_stride + p.hist_off;
         if (r == 0 || at.known == 0) walk.begin(p, x, row, at.known, hist, c);
         float u[8], y[8];
@@ -492,7 +505,7 @@ __global__ void __launch_bounds__(VEC_THREADS) conv_heads_vec_kernel(ConvArgs p)
                 const unsigned lanes = LANES == 32 ? 0xffffffffu : ((1u << LANES) - 1u) << ((threadIdx.x & 31) / LANES * LANES);
 #pragma unroll
                 for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(lanes, ss, o);
-                const float inv = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
+                const float inv = inverse_rms<T>(fmaf(ss, inv_dim, p.eps));
 #pragma unroll
                 for (int i = 0; i < 8; ++i) y[i] *= inv;
             }
@@ -500,9 +513,8 @@ __global__ void __launch_bounds__(VEC_THREADS) conv_heads_vec_kernel(ConvArgs p)
         if (is_q) {
             store_eight((T*)p.q_out + (size_t)row * nq + c, y);
         } else {
-            const size_t to = (size_t)p.block_table[(size_t)at.seq * p.table_width + at.pos / PAGE_ROWS] * PAGE_ROWS + at.pos % PAGE_ROWS;
-            if (is_v) store_eight((T*)p.v_pool + to * nv + (c - nq - nk), y);
-            else store_eight((T*)p.k_pool + to * nk + (c - nq), y);
+            if (is_v) store_eight((T*)p.v_pool + (size_t)at.to * nv + (c - nq - nk), y);
+            else store_eight((T*)p.k_pool + (size_t)at.to * nk + (c - nq), y);
         }
     }
 }
@@ -527,8 +539,9 @@ __global__ void __launch_bounds__(VEC_THREADS) conv_rows_vec_kernel(ConvArgs p) 
     const int row0 = blockIdx.x * R, n = min(R, p.rows - row0);
     const int c = 8 * (blockIdx.y * VEC_THREADS + threadIdx.x);
     const bool live = c < p.channels;
+    __shared__ RowPlace place[R];
     Walk<TI> walk;
-    const RowPlace first = place_of(p, row0);
+    if ((int)threadIdx.x < n) place[threadIdx.x] = place_of(p, row0 + threadIdx.x);
     float bias[8];
     if (live) {
         walk.load_taps(p, c);
@@ -537,6 +550,7 @@ __global__ void __launch_bounds__(VEC_THREADS) conv_rows_vec_kernel(ConvArgs p) 
     }
     fr_pdl_wait();
     fr_pdl_launch();
+    __syncthreads();
     if (!live) return;
     const TI* x = (const TI*)p.x;
     Eight<TI> raw[R];
@@ -547,8 +561,8 @@ __global__ void __launch_bounds__(VEC_THREADS) conv_rows_vec_kernel(ConvArgs p) 
     for (int r = 0; r < R; ++r) {
         if (r >= n) break;
         const int row = row0 + r;
-        const RowPlace at = r == 0 ? first : place_of(p, row);
-        if (at.seq < 0) continue;
+        const RowPlace at = place[r];
+        if (at.known < 0) continue;
         float* hist = p.state + (size_t)at.slot * p.state_stride + p.hist_off;
         if (r == 0 || at.known == 0) walk.begin(p, x, row, at.known, hist, c);
         float u[8], y[8];

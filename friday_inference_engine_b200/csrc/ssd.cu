@@ -12,7 +12,7 @@
 //                  memory.  A one-token step is the same kernel: all of a block's state is requested at once.
 //   chunk_states   bf16 prompts, on the tensor cores (mma.sync.m16n8k16, fp32 sums): a prompt is cut into chunks of 128 tokens; with
 //                  c_t the sum of the decays' logarithms up to token t of its chunk, a chunk adds U = sum_t e^(c_last - c_t) dt_t B_t x_t^T
-//                  to e^(c_last) times the state before it.  The scaled B enter the product as two bf16 numbers each (head and
+//                  to e^(c_last) times the state before it.  The scaled x enter the product as two bf16 numbers each (head and
 //                  remainder), which keeps them 32-bit in effect.
 //   chunk_chain    walks a sequence's chunks in order, fp32: leaves every chunk's starting state where its U was and the last
 //                  state with the sequence.
@@ -122,36 +122,32 @@ constexpr int THR = 256;            // threads of a chunk's block
 constexpr int WARPS = THR / 32;
 static_assert(WARPS * 16 == CH, "a warp owns sixteen of a chunk's tokens");
 
-// Warp 0: the step sizes of a chunk's tokens, and the running sums of the decays' logarithms (in units of log2), the last of them at [CH]
+// The step sizes of a chunk's tokens, and the running sums of the decays' logarithms (in units of log2), the last of them at [CH]; a thread
+// per token, then a barrier
 __device__ __forceinline__ void chunk_steps(const SsdArgs& p, int r0, int n, int head, float* step, float* cum) {
-    if (threadIdx.x >= 32) return;
-    constexpr int PER = CH / 32;
-    const int lane = threadIdx.x;
-    const float rate = -LOG2E * expf(p.a_log.at(head));
-    float dt[PER], own[PER], sum = 0.f;
+    __shared__ float sums[CH / 32];
+    const int t = threadIdx.x, lane = t & 31, warp = t >> 5;
+    float dt = 0.f, sum = 0.f;
+    if (t < CH) {
+        dt = t < n ? step_of(p, r0 + t, head) : 0.f;
+        sum = -LOG2E * expf(p.a_log.at(head)) * dt;
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        const int t = lane * PER + i;
-        dt[i] = t < n ? step_of(p, r0 + t, head) : 0.f;
+        for (int o = 1; o < 32; o <<= 1) {
+            const float v = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += v;
+        }
+        if (lane == 31) sums[warp] = sum;
+        step[t] = dt;
     }
+    __syncthreads();
+    if (t < CH) {
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        sum += rate * dt[i];
-        own[i] = sum;
+        for (int w = 0; w < CH / 32; ++w)
+            if (w < warp) sum += sums[w];
+        cum[t] = sum;
+        if (t == CH - 1) cum[CH] = sum;
     }
-    float before = sum;                                        // an inclusive sum over the lanes, then without the lane's own
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-        const float v = __shfl_up_sync(0xffffffffu, before, o);
-        if (lane >= o) before += v;
-    }
-    before -= sum;
-#pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        step[lane * PER + i] = dt[i];
-        cum[lane * PER + i] = before + own[i];
-    }
-    if (lane == 31) cum[CH] = before + sum;
+    __syncthreads();
 }
 
 // A thread's share of the rows r0 .. r0 + n - 1 of `width` channels: all loads first (`fetch`), stored to a tile [CH][D + PAD] later
@@ -177,10 +173,10 @@ __device__ __forceinline__ void put_rows(const uint4 (&raw)[pieces_of<D>()], bf1
 template <int DK, int DV>
 __global__ void __launch_bounds__(THR) chunk_states_kernel(SsdArgs p) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    bf16* sbh = (bf16*)smem_raw;                          // [CH][DK + PAD] scaled B, head
-    bf16* sbl = sbh + CH * (DK + PAD);                    // and remainder
-    bf16* sx = sbl + CH * (DK + PAD);                     // [CH][DV + PAD]
-    __shared__ float step[CH], cum[CH + 1];
+    bf16* sb = (bf16*)smem_raw;                           // [CH][DK + PAD]
+    bf16* sxh = sb + CH * (DK + PAD);                     // [CH][DV + PAD] scaled x, head
+    bf16* sxl = sxh + CH * (DV + PAD);                    // and remainder
+    __shared__ __align__(8) float step[CH], cum[CH + 2];
     // warps share the tiles of 16 rows of the state; where there are fewer tiles than warps, the value channels as well
     constexpr int MT = DK / 16, COLS = WARPS / MT, DVW = DV / COLS < 16 ? 16 : DV / COLS;
     static_assert(MT <= WARPS, "at most eight tiles of the state's rows");
@@ -194,23 +190,22 @@ __global__ void __launch_bounds__(THR) chunk_states_kernel(SsdArgs p) {
     if (p.row_seq[r0] < 0) return;
     const int bg = head / (p.heads / p.groups);
     uint4 br[pieces_of<DK>()], xr[pieces_of<DV>()];
-    fetch_rows<DK>(p, p.b_off + bg * p.n, p.n, r0, n, br);
     fetch_rows<DV>(p, p.x_off + head * p.dv, p.dv, r0, n, xr);
+    fetch_rows<DK>(p, p.b_off + bg * p.n, p.n, r0, n, br);
     chunk_steps(p, r0, n, head, step, cum);
-    __syncthreads();
     if (threadIdx.x == 0) p.chunk_decay[((size_t)seq * p.max_chunks + c) * p.heads + head] = exp2f(cum[CH]);
 #pragma unroll
-    for (int i = 0; i < pieces_of<DK>(); ++i) {
-        const int idx = threadIdx.x + i * THR, t = idx / (DK / 8), k = (idx % (DK / 8)) * 8;
+    for (int i = 0; i < pieces_of<DV>(); ++i) {
+        const int idx = threadIdx.x + i * THR, t = idx / (DV / 8), k = (idx % (DV / 8)) * 8;
         const float f = exp2f(cum[CH] - cum[t]) * step[t];          // zero beyond the last token
-        const uint32_t w[4] = {br[i].x, br[i].y, br[i].z, br[i].w};
+        const uint32_t w[4] = {xr[i].x, xr[i].y, xr[i].z, xr[i].w};
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) split2(__uint_as_float(w[e] << 16) * f, __uint_as_float(w[e] & 0xffff0000u) * f, hi[e], lo[e]);
-        *(uint4*)(sbh + t * (DK + PAD) + k) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        *(uint4*)(sbl + t * (DK + PAD) + k) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        *(uint4*)(sxh + t * (DV + PAD) + k) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *(uint4*)(sxl + t * (DV + PAD) + k) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
-    put_rows<DV>(xr, sx);
+    put_rows<DK>(br, sb);
     __syncthreads();
     const int m0 = warp % MT, v0 = (warp / MT) * DVW;
     if (v0 >= DV) return;
@@ -221,17 +216,18 @@ __global__ void __launch_bounds__(THR) chunk_states_kernel(SsdArgs p) {
 #pragma unroll
     for (int ks = 0; ks < CH / 16; ++ks) {
         if (ks * 16 >= n) break;
-        uint32_t ah[4], al[4];
-        ldsm4t(ah, sbh + (ks * 16 + a_row) * (DK + PAD) + m0 * 16 + a_col);
-        ldsm4t(al, sbl + (ks * 16 + a_row) * (DK + PAD) + m0 * 16 + a_col);
+        uint32_t a[4];
+        ldsm4t(a, sb + (ks * 16 + a_row) * (DK + PAD) + m0 * 16 + a_col);
 #pragma unroll
         for (int j = 0; j < DVW / 16; ++j) {
-            uint32_t b[4];
-            ldsm4t(b, sx + (ks * 16 + (lane & 15)) * (DV + PAD) + v0 + j * 16 + (lane >> 4) * 8);
-            mma_16816(acc[2 * j], ah, b[0], b[1]);
-            mma_16816(acc[2 * j], al, b[0], b[1]);
-            mma_16816(acc[2 * j + 1], ah, b[2], b[3]);
-            mma_16816(acc[2 * j + 1], al, b[2], b[3]);
+            uint32_t bh[4], bl[4];
+            const int at = (ks * 16 + (lane & 15)) * (DV + PAD) + v0 + j * 16 + (lane >> 4) * 8;
+            ldsm4t(bh, sxh + at);
+            ldsm4t(bl, sxl + at);
+            mma_16816(acc[2 * j], a, bh[0], bh[1]);
+            mma_16816(acc[2 * j + 1], a, bh[2], bh[3]);
+            mma_16816(acc[2 * j], a, bl[0], bl[1]);
+            mma_16816(acc[2 * j + 1], a, bl[2], bl[3]);
         }
     }
     float* U = p.chunk + (((size_t)seq * p.max_chunks + c) * p.heads + head) * p.n * p.dv;
@@ -307,7 +303,7 @@ __global__ void __launch_bounds__(THR) chunk_outputs_kernel(SsdArgs p) {
     bf16* sl = sh + DK * (DV + PAD);                      // and remainder; once they are used, in their place:
     bf16* sb = sh;                                        // [CH][DK + PAD]
     bf16* sx = sb + CH * (DK + PAD);                      // [CH][DV + PAD]
-    __shared__ float step[CH], cum[CH + 1];
+    __shared__ __align__(8) float step[CH], cum[CH + 2];
     const int c = blockIdx.x, head = blockIdx.y, seq = blockIdx.z;
     const int qlen = p.seq_qlen[seq];
     if (c * CH >= qlen) return;
@@ -376,8 +372,8 @@ __global__ void __launch_bounds__(THR) chunk_outputs_kernel(SsdArgs p) {
                 ldsm4t(bh, sh + (ks * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
                 ldsm4t(bl, sl + (ks * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
                 mma_16816(o[2 * j], ca, bh[0], bh[1]);
-                mma_16816(o[2 * j], ca, bl[0], bl[1]);
                 mma_16816(o[2 * j + 1], ca, bh[2], bh[3]);
+                mma_16816(o[2 * j], ca, bl[0], bl[1]);
                 mma_16816(o[2 * j + 1], ca, bl[2], bl[3]);
             }
         }
@@ -397,41 +393,50 @@ __global__ void __launch_bounds__(THR) chunk_outputs_kernel(SsdArgs p) {
     put_rows<DV>(xr, sx);
     __syncthreads();
     if (!mine) return;
-    // and the chunk's own tokens, those up to each row (a warp's rows see no token beyond its last row)
+    // and the chunk's own tokens, those up to each row (a warp's rows see no token beyond its last row), 32 at a time: four sums run side
+    // by side
 #pragma unroll 1
-    for (int kk = 0; kk <= warp; ++kk) {
-        float s[2][4];
+    for (int kk = 0; kk <= warp; kk += 2) {
+        float s[4][4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[0][e] = s[1][e] = 0.f;
+        for (int nt = 0; nt < 4; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+        const bf16* b_at = sb + (kk * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * (DK + PAD) + ((lane >> 3) & 1) * 8;      // stored [token][channel]
 #pragma unroll
         for (int ks = 0; ks < DK / 16; ++ks) {
-            uint32_t ca[4], b[4];                         // tokens kk * 16 .. + 15: the second operand is stored [token][channel]
+            uint32_t ca[4], b0[4], b1[4];
             ldsm4(ca, c_at + ks * 16);
-            ldsm4(b, sb + (kk * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * (DK + PAD) + ks * 16 + ((lane >> 3) & 1) * 8);
-            mma_16816(s[0], ca, b[0], b[1]);
-            mma_16816(s[1], ca, b[2], b[3]);
+            ldsm4(b0, b_at + ks * 16);
+            ldsm4(b1, b_at + 16 * (DK + PAD) + ks * 16);
+            mma_16816(s[0], ca, b0[0], b0[1]);
+            mma_16816(s[1], ca, b0[2], b0[3]);
+            mma_16816(s[2], ca, b1[0], b1[1]);
+            mma_16816(s[3], ca, b1[2], b1[3]);
         }
+        uint32_t hi[2][4], lo[2][4];
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
+        for (int nt = 0; nt < 4; ++nt) {
+            const int t = kk * 16 + nt * 8 + 2 * t4;
+            const float2 ct = *(const float2*)(cum + t), st = *(const float2*)(step + t);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int t = kk * 16 + nt * 8 + 2 * t4 + (e & 1);
-                s[nt][e] = t <= row[e >> 1] ? s[nt][e] * (exp2f(at[e >> 1] - cum[t]) * step[t]) : 0.f;
+                const int half = e >> 1;
+                const float f = exp2f(at[half] - (e & 1 ? ct.y : ct.x)) * (e & 1 ? st.y : st.x);
+                s[nt][e] = t + (e & 1) <= row[half] ? s[nt][e] * f : 0.f;
             }
-        uint32_t hi[4], lo[4];
-        split2(s[0][0], s[0][1], hi[0], lo[0]);
-        split2(s[0][2], s[0][3], hi[1], lo[1]);
-        split2(s[1][0], s[1][1], hi[2], lo[2]);
-        split2(s[1][2], s[1][3], hi[3], lo[3]);
-#pragma unroll
-        for (int j = 0; j < DV / 16; ++j) {
-            uint32_t b[4];
-            ldsm4t(b, sx + (kk * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
-            mma_16816(o[2 * j], hi, b[0], b[1]);
-            mma_16816(o[2 * j], lo, b[0], b[1]);
-            mma_16816(o[2 * j + 1], hi, b[2], b[3]);
-            mma_16816(o[2 * j + 1], lo, b[2], b[3]);
+            split2(s[nt][0], s[nt][1], hi[nt >> 1][2 * (nt & 1)], lo[nt >> 1][2 * (nt & 1)]);
+            split2(s[nt][2], s[nt][3], hi[nt >> 1][2 * (nt & 1) + 1], lo[nt >> 1][2 * (nt & 1) + 1]);
         }
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int j = 0; j < DV / 16; ++j) {
+                uint32_t b[4];
+                ldsm4t(b, sx + ((kk + u) * 16 + (lane & 15)) * (DV + PAD) + j * 16 + (lane >> 4) * 8);
+                mma_16816(o[2 * j], hi[u], b[0], b[1]);
+                mma_16816(o[2 * j + 1], hi[u], b[2], b[3]);
+                mma_16816(o[2 * j], lo[u], b[0], b[1]);
+                mma_16816(o[2 * j + 1], lo[u], b[2], b[3]);
+            }
     }
     const bool pairs = p.dv % 2 == 0;
     const float skip = p.skip.at(head);
@@ -455,7 +460,7 @@ __global__ void __launch_bounds__(THR) chunk_outputs_kernel(SsdArgs p) {
 
 template <int DK, int DV>
 int launch_chunks(const SsdArgs& p, int n_seqs, cudaStream_t stream) {
-    constexpr int smem_a = (2 * CH * (DK + PAD) + CH * (DV + PAD)) * 2, smem_c = outputs_smem<DK, DV>();
+    constexpr int smem_a = (CH * (DK + PAD) + 2 * CH * (DV + PAD)) * 2, smem_c = outputs_smem<DK, DV>();
     static bool set = false;
     if (!set) {
         FR_CUDA(cudaFuncSetAttribute(chunk_states_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_a));
